@@ -365,6 +365,106 @@ int b2kv_matmul(const void* a, const void* w, const void* bias, const void* resi
                 int activation, int dtype, int32_t* dev_status, void* stream);
 
 /*
+ * Building blocks of decoders with a 32-bit residual stream (RMS norms, gated feed-forwards, latent attention, mixtures
+ * of experts).  No counterpart in the reference, whose decoder is the LayerNorm / GELU block above.  `dtype` is the
+ * storage type of activations and weights; norms, rotations, scores, routers and the residual are computed in 32-bit.
+ */
+
+/* out[i, :] = table[ids[i], :] in fp32 (the start of a 32-bit residual stream; no position is added).  A token id outside
+ * the table is clamped and recorded in dev_status. */
+int b2kv_embed_rows(const void* table, const int32_t* ids, float* out, int rows, int dim, int vocab, int dtype,
+                    int32_t* dev_status, void* stream);
+
+/* out[i, :] = x[r, :] / sqrt(mean(x[r, :]^2) + eps) * (w + w_offset), r = row_index ? row_index[i] : i; x and w fp32, out
+ * of `dtype`.  w_offset = 1 is the form whose weights are stored around zero. */
+int b2kv_rmsnorm(const float* x, int64_t ld_x, const int32_t* row_index, const float* w, float w_offset, void* out,
+                 int64_t ld_out, int rows, int size, float eps, int dtype, void* stream);
+
+/*
+ * out = x @ w per group, with the output columns cut into up to three segments that go to places of their own:
+ *   B2KV_SEG_STORE      the product, in the storage type
+ *   B2KV_SEG_F32        the product (+ residual), fp32: the residual stream, router scores, logits
+ *   B2KV_SEG_GLU_SILU   columns come in pairs (gate, up): silu(gate) * up, half as many output columns
+ *   B2KV_SEG_GLU_CLAMP  pairs (gate, up): g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1)
+ * x is [rows, K] with row pitch ld_x; w is [K, N] row-major with row pitch ld_w.  Group g (0 <= g < groups) reads
+ * x + g * group_x and w + g * group_w and writes seg.out + g * seg.group: the heads of a per-head product.  With group_rows
+ * (device, groups + 1 row offsets) group g instead owns rows group_rows[g] .. group_rows[g + 1] - 1 of x and of the outputs:
+ * the experts of a mixture, whose rows are sorted by expert; no group has more than max_group_rows of them.
+ * Offsets and pitches are in elements.  Segment boundaries are even.  The product runs on the tensor cores for bf16 when
+ * pitches, offsets and boundaries allow it (multiples of 8 elements; boundaries multiples of 32): at most 128 rows per
+ * group stream the weights once, more go to the tiled kernel; everything else, and fp32, runs on a CUDA-core kernel.
+ * path: 0 = choose, 1 = CUDA cores, 2 = weight streaming, 3 = tiled (refused when the shape is not one it takes).
+ */
+#define B2KV_SEG_STORE 0
+#define B2KV_SEG_F32 1
+#define B2KV_SEG_GLU_SILU 2
+#define B2KV_SEG_GLU_CLAMP 3
+#define B2KV_MAX_SEGMENTS 3
+typedef struct b2kv_segment {
+    void* out;
+    int64_t ld, group; /* row pitch of out; offset between groups */
+    int32_t end, kind; /* first column (of w) behind the segment */
+} b2kv_segment;
+typedef struct b2kv_linear_args {
+    const void* x;
+    const void* w;
+    const float* residual; /* added to fp32 segments (may be the output itself), or NULL */
+    const int32_t* group_rows;
+    int64_t ld_x, group_x, ld_w, group_w, ld_residual;
+    b2kv_segment seg[B2KV_MAX_SEGMENTS];
+    int32_t rows, K, N, groups, max_group_rows, n_seg, dtype, path;
+    float limit;
+} b2kv_linear_args;
+int b2kv_linear(const b2kv_linear_args* args, int32_t* dev_status, void* stream);
+
+/*
+ * Latent attention (one latent row and one rotated key part per token, shared by all heads, are what the cache holds).
+ * b2kv_latent_append, per row i of y at position row_pos[i] of sequence row_slot[i] (row_slot NULL: sequence i):
+ *   - rotates the last `rot` of every head's dim + rot query elements in place (heads from column 0 on);
+ *   - with latent_cache: columns [down_col, down_col + kv_rank) are RMS-normed with w_norm and eps and stored as the latent
+ *     row, the next `rot` are rotated and stored as the key part.  latent_cache [sequences * T_max, kv_rank], key_cache
+ *     [sequences * T_max, rot].
+ * The rotation pairs element j with j + rot_dims / 2 of the first rot_dims elements and turns them by position *
+ * inv_freq[j]; elements past rot_dims pass.  A position outside [0, T_max) is skipped and recorded in dev_status.
+ */
+int b2kv_latent_append(void* y, int64_t ld_y, int H, int dim, int rot, int rot_dims, const float* inv_freq, int down_col,
+                       int kv_rank, const float* w_norm, float eps, void* key_cache, void* latent_cache,
+                       const int32_t* row_slot, const int32_t* row_pos, int n_slots, int T_max, int rows, int dtype,
+                       int32_t* dev_status, void* stream);
+
+/*
+ * Attention of single query rows over the cached latent rows, in the latent space: per row i and head h
+ *   score_t = (q_latent[i, h, :] . latent[t, :] + q[i, h, dim:] . key[t, :]) * scale,  t in (row_pos[i] - window, row_pos[i]]
+ *   out[i, h, :] = sum_t softmax(score)_t latent[t, :]
+ * q_latent [rows, H, kv_rank] is the unrotated query carried into the latent space; window <= 0 sees every earlier token.
+ * span is an upper bound of the tokens a row sees.  The rows' own tokens are in the cache already.  bf16 with kv_rank a
+ * multiple of 64 up to 512, rot a multiple of 16 up to 64 and H up to 128 runs on the tensor cores (split over the window, partial results
+ * merged by the CTA that finishes a row last; workspace of b2kv_latent_decode_workspace_bytes bytes, zeroed once before
+ * its first use), everything else on CUDA cores.  path: 0 = choose, 1 = CUDA cores, 2 = tensor cores.
+ */
+size_t b2kv_latent_decode_workspace_bytes(int rows, int H, int kv_rank, int span, int dtype);
+int b2kv_latent_decode(const void* q_latent, const void* q, int64_t ld_q, int dim, const void* key_cache,
+                       const void* latent_cache, void* out, const int32_t* row_slot, const int32_t* row_pos, int n_slots,
+                       int T_max, int rows, int H, int kv_rank, int rot, int window, int span, float scale, int dtype,
+                       int path, void* workspace, size_t workspace_bytes, int32_t* dev_status, void* stream);
+
+/*
+ * Mixture of experts.  b2kv_route: per row of logits [rows, ld] (fp32, `experts` of them used): softmax over all experts,
+ * the `keep` best of `groups` equal groups by their largest score, the `top` best experts of those (lowest index among
+ * equals); expert ids and scores go to idx / score [rows, top], and the experts' row counts to counts (int32[2 * experts]:
+ * the counts, then working counters of b2kv_moe_plan that this call sets to zero).  experts up to 1024, top up to 64.
+ * b2kv_moe_plan sorts the rows * top choices by expert: offsets (int32[experts + 1]) and slot [rows, top] (the sorted place
+ * of every choice), and copies every row of h to its sorted places: sorted [rows * top, dim].
+ * b2kv_moe_combine: x[i, :] += sum_k score[i, k] * y[slot[i, k], :] (x fp32, y of `dtype`).
+ */
+int b2kv_route(const float* logits, int64_t ld, int rows, int experts, int groups, int keep, int top, int32_t* idx,
+               float* score, int32_t* counts, void* stream);
+int b2kv_moe_plan(const int32_t* idx, int32_t* counts, int rows, int experts, int top, int32_t* offsets, int32_t* slot,
+                  const void* h, int64_t ld_h, void* sorted, int64_t ld_sorted, int dim, int dtype, void* stream);
+int b2kv_moe_combine(float* x, int64_t ld_x, const void* y, int64_t ld_y, const int32_t* slot, const float* score, int rows,
+                     int top, int dim, int dtype, void* stream);
+
+/*
  * Tuning hook for experiments (process-global and unsynchronised: set knobs before launching work, never while
  * another thread is inside a b2kv call): sets an integer knob by name ("decode_variant",
  * "decode_grid_per_sm", "decode_l2_keep", "decode_no_tensor_map", "decode_dynamic_chunks": small chunks of the

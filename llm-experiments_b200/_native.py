@@ -34,6 +34,28 @@ _i = ctypes.c_int
 _i64 = ctypes.c_int64
 _sz = ctypes.c_size_t
 
+_f = ctypes.c_float
+
+SEG_STORE, SEG_F32, SEG_GLU_SILU, SEG_GLU_CLAMP = 0, 1, 2, 3
+MAX_SEGMENTS = 3
+
+
+class Segment(ctypes.Structure):
+    """``b2kv_segment``: where a range of output columns of a linear layer goes."""
+
+    _fields_ = [("out", _vp), ("ld", _i64), ("group", _i64), ("end", ctypes.c_int32), ("kind", ctypes.c_int32)]
+
+
+class LinearArgs(ctypes.Structure):
+    """``b2kv_linear_args``."""
+
+    _fields_ = [("x", _vp), ("w", _vp), ("residual", _vp), ("group_rows", _vp), ("ld_x", _i64), ("group_x", _i64),
+                ("ld_w", _i64), ("group_w", _i64), ("ld_residual", _i64), ("seg", Segment * MAX_SEGMENTS),
+                ("rows", ctypes.c_int32), ("K", ctypes.c_int32), ("N", ctypes.c_int32), ("groups", ctypes.c_int32),
+                ("max_group_rows", ctypes.c_int32), ("n_seg", ctypes.c_int32), ("dtype", ctypes.c_int32),
+                ("path", ctypes.c_int32), ("limit", _f)]
+
+
 # name -> (restype, argtypes); kept in the order of include/b2kv.h
 SIGNATURES = {
     "b2kv_strerror": (ctypes.c_char_p, [_i]),
@@ -73,6 +95,16 @@ SIGNATURES = {
     "b2kv_qkv_append": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i64, _i64, _i64, _i, _vp, _vp]),
     "b2kv_matmul_rows": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp]),
     "b2kv_matmul": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp]),
+    "b2kv_embed_rows": (_i, [_vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp]),
+    "b2kv_rmsnorm": (_i, [_vp, _i64, _vp, _vp, _f, _vp, _i64, _i, _i, _f, _i, _vp]),
+    "b2kv_linear": (_i, [ctypes.POINTER(LinearArgs), _vp, _vp]),
+    "b2kv_latent_append": (_i, [_vp, _i64, _i, _i, _i, _i, _vp, _i, _i, _vp, _f, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp]),
+    "b2kv_latent_decode_workspace_bytes": (_sz, [_i, _i, _i, _i, _i]),
+    "b2kv_latent_decode": (_i, [_vp, _vp, _i64, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp,
+                                _sz, _vp, _vp]),
+    "b2kv_route": (_i, [_vp, _i64, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp]),
+    "b2kv_moe_plan": (_i, [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _i64, _vp, _i64, _i, _i, _vp]),
+    "b2kv_moe_combine": (_i, [_vp, _i64, _vp, _i64, _vp, _vp, _i, _i, _i, _i, _vp]),
     "b2kv_tune": (_i, [ctypes.c_char_p, _i]),
 }
 

@@ -1,0 +1,136 @@
+// b2kv_linear: argument checks, the choice of the kernel, and the CUDA-core kernel for fp32 and for shapes that the
+// tensor-core kernels do not take (64 x 64 output tiles, 16 input features per step, 4 x 4 outputs per thread, fp32
+// accumulation).
+#include "linear.cuh"
+
+namespace b2kv {
+namespace lin {
+
+constexpr int kTile = 64, kStep = 16, kThreads = 256;
+
+// Exact exponential for the fp32 path; the bf16 paths round the result to 8 bits anyway.
+template <typename T>
+__device__ __forceinline__ float glu_value(int kind, float g, float u, float limit) {
+    if (sizeof(T) == 2) return glu(kind, g, u, limit);
+    if (kind == B2KV_SEG_GLU_SILU) return g / (1.0f + expf(-g)) * u;
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads) linear_simt_kernel(const b2kv_linear_args a) {
+    __shared__ float xs[kStep][kTile + 4];
+    __shared__ float ws[kStep][kTile + 4];
+    const int g = blockIdx.z;
+    int first = 0, n_rows = a.rows;
+    const T* x = static_cast<const T*>(a.x);
+    if (a.group_rows != nullptr) {
+        first = a.group_rows[g];
+        n_rows = a.group_rows[g + 1] - first;
+        x += static_cast<int64_t>(first) * a.ld_x;
+    } else {
+        x += static_cast<int64_t>(g) * a.group_x;
+    }
+    const int row0 = blockIdx.y * kTile, col0 = blockIdx.x * kTile;
+    if (row0 >= n_rows) return;
+    const T* w = static_cast<const T*>(a.w) + static_cast<int64_t>(g) * a.group_w;
+    const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < a.K; k0 += kStep) {
+        for (int i = threadIdx.x; i < kTile * kStep; i += kThreads) {
+            const int r = i / kStep, k = i % kStep;
+            xs[k][r] = (row0 + r < n_rows && k0 + k < a.K)
+                           ? Elt<T>::to_float(x[static_cast<int64_t>(row0 + r) * a.ld_x + k0 + k]) : 0.f;
+            const int wk = i / kTile, c = i % kTile;
+            ws[wk][c] = (k0 + wk < a.K && col0 + c < a.N)
+                            ? Elt<T>::to_float(w[static_cast<int64_t>(k0 + wk) * a.ld_w + col0 + c]) : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < kStep; ++k) {
+            float xv[4], wv[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) xv[i] = xs[k][ty * 4 + i], wv[i] = ws[k][tx * 4 + i];
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xv[i], wv[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int r = row0 + ty * 4 + i;
+        if (r >= n_rows) break;
+        const int64_t out_row = first + r;
+#pragma unroll
+        for (int j = 0; j < 4; j += 2) {  // pairs of columns: boundaries of segments are even
+            const int c = col0 + tx * 4 + j;
+            if (c >= a.N) break;
+            const int s = segment_of(a, c);
+            const b2kv_segment& sg = a.seg[s];
+            const int local = c - segment_first(a, s);
+            const int64_t base = out_row * sg.ld + static_cast<int64_t>(g) * (a.group_rows ? 0 : sg.group);
+            if (sg.kind >= B2KV_SEG_GLU_SILU) {
+                static_cast<T*>(sg.out)[base + local / 2] =
+                    Elt<T>::from_float(glu_value<T>(sg.kind, acc[i][j], acc[i][j + 1], a.limit));
+                continue;
+            }
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                if (c + e >= a.N) break;
+                float v = acc[i][j + e];
+                if (sg.kind == B2KV_SEG_F32) {
+                    if (a.residual != nullptr) v += a.residual[out_row * a.ld_residual + local + e];
+                    static_cast<float*>(sg.out)[base + local + e] = v;
+                } else {
+                    static_cast<T*>(sg.out)[base + local + e] = Elt<T>::from_float(v);
+                }
+            }
+        }
+    }
+}
+
+static int launch_simt(const b2kv_linear_args& a, void* stream) {
+    const int max_rows = a.group_rows ? a.max_group_rows : a.rows;
+    const dim3 grid((a.N + kTile - 1) / kTile, (max_rows + kTile - 1) / kTile, a.groups);
+    if (grid.y > 65535u || grid.z > 65535u) return B2KV_ERR_UNSUPPORTED;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (a.dtype == B2KV_DTYPE_F32)
+        linear_simt_kernel<float><<<grid, kThreads, 0, s>>>(a);
+    else
+        linear_simt_kernel<__nv_bfloat16><<<grid, kThreads, 0, s>>>(a);
+    B2KV_CUDA_TRY(cudaGetLastError());
+    return B2KV_OK;
+}
+
+}  // namespace lin
+}  // namespace b2kv
+
+using namespace b2kv;
+
+extern "C" int b2kv_linear(const b2kv_linear_args* args, int32_t* dev_status, void* stream) {
+    if (args == nullptr) return B2KV_ERR_BAD_ARG;
+    const b2kv_linear_args& a = *args;
+    if (elt_bytes(a.dtype) == 0) return B2KV_ERR_UNSUPPORTED;
+    if (!a.x || !a.w || a.rows <= 0 || a.K <= 0 || a.N <= 0 || a.groups <= 0 || a.path < 0 || a.path > 3) return B2KV_ERR_BAD_ARG;
+    if (a.n_seg < 1 || a.n_seg > B2KV_MAX_SEGMENTS || a.seg[a.n_seg - 1].end != a.N) return B2KV_ERR_BAD_ARG;
+    if (a.group_rows && (a.max_group_rows <= 0 || a.max_group_rows > a.rows)) return B2KV_ERR_BAD_ARG;
+    int first = 0;
+    for (int s = 0; s < a.n_seg; ++s) {
+        const b2kv_segment& sg = a.seg[s];
+        if (!sg.out || sg.end <= first || sg.kind < B2KV_SEG_STORE || sg.kind > B2KV_SEG_GLU_CLAMP) return B2KV_ERR_BAD_ARG;
+        // pairs of columns never straddle a boundary (the last segment may end on an odd column if it has no pairs)
+        if ((sg.end & 1) && (s + 1 < a.n_seg || sg.kind >= B2KV_SEG_GLU_SILU)) return B2KV_ERR_BAD_ARG;
+        first = sg.end;
+    }
+    if (a.path == 2) return linear_rows_tc(a, dev_status, stream);
+    if (a.path == 3) return linear_tiled_tc(a, dev_status, stream);
+    if (a.path == 0 && a.dtype == B2KV_DTYPE_BF16) {
+        const int rc = (a.group_rows ? a.max_group_rows : a.rows) <= 128 ? linear_rows_tc(a, dev_status, stream)
+                                                                         : linear_tiled_tc(a, dev_status, stream);
+        if (rc != B2KV_ERR_UNSUPPORTED) return rc;
+    }
+    return lin::launch_simt(a, stream);
+}

@@ -1,0 +1,32 @@
+// Grouped, segmented linear layers (b2kv_linear): what the three kernels behind the entry point share.
+#pragma once
+
+#include "b2kv_common.cuh"
+
+namespace b2kv {
+namespace lin {
+
+// x * sigmoid(1.702 x) of the clamped gate times the clamped up part plus one; silu(gate) * up.
+__device__ __forceinline__ float glu(int kind, float g, float u, float limit) {
+    if (kind == B2KV_SEG_GLU_SILU) return g / (1.0f + __expf(-g)) * u;
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+}
+
+// Index of the segment that holds column c (segments are in column order).
+__device__ __forceinline__ int segment_of(const b2kv_linear_args& a, int c) {
+    int s = 0;
+    while (s + 1 < a.n_seg && c >= a.seg[s].end) ++s;
+    return s;
+}
+
+__device__ __forceinline__ int segment_first(const b2kv_linear_args& a, int s) { return s == 0 ? 0 : a.seg[s - 1].end; }
+
+}  // namespace lin
+
+// bf16 kernels on the tensor cores; B2KV_ERR_UNSUPPORTED when the shape is not one they take.
+int linear_rows_tc(const b2kv_linear_args& a, int32_t* dev_status, void* stream);   // linear_rows.cu
+int linear_tiled_tc(const b2kv_linear_args& a, int32_t* dev_status, void* stream);  // gemm.cu
+
+}  // namespace b2kv

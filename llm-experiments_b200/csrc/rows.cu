@@ -1,0 +1,122 @@
+// Row operations around a 32-bit residual stream: the token rows that start it, and RMS norms that read it.
+// These kernels may be scheduled ahead of the end of the kernel that writes their inputs, so no pointer to such data is
+// const __restrict__: the compiler would take it for data that nothing writes and could load it before the wait.
+#include "b2kv_common.cuh"
+
+namespace b2kv {
+namespace {
+
+constexpr int kThreads = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads) embed_rows_kernel(const T* table, const int32_t* ids,
+                                                              float* out, int dim, int vocab, int32_t* dev_status) {
+    grid_launch_dependents();
+    if (threadIdx.x == 0) grid_dependency_wait();
+    __syncthreads();
+    int id = ids[blockIdx.x];
+    if (id < 0 || id >= vocab) {
+        if (threadIdx.x == 0) report_status(dev_status, B2KV_DEV_BAD_TOKEN);
+        id = id < 0 ? 0 : vocab - 1;
+    }
+    const T* src = table + static_cast<int64_t>(id) * dim;
+    float* dst = out + static_cast<int64_t>(blockIdx.x) * dim;
+    for (int i = threadIdx.x; i < dim; i += kThreads) dst[i] = Elt<T>::to_float(src[i]);
+}
+
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&lo);
+    u.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = u;
+}
+
+// One CTA per row; a row of up to 16384 elements stays in registers between the two passes.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) rmsnorm_kernel(const float* x, int64_t ld_x,
+                                                           const int32_t* row_index, const float* w,
+                                                           float w_offset, T* out, int64_t ld_out, int size,
+                                                           float eps, bool vec) {
+    constexpr int kKeep = 16;
+    __shared__ float part[kThreads / 32];
+    grid_launch_dependents();
+    if (threadIdx.x == 0) grid_dependency_wait();
+    __syncthreads();
+    const int64_t row = row_index ? row_index[blockIdx.x] : static_cast<int>(blockIdx.x);
+    const float* xr = x + row * ld_x;
+    T* yr = out + static_cast<int64_t>(blockIdx.x) * ld_out;
+    const int chunks = vec ? size / 4 : 0;
+    float4 keep[kKeep];
+    float sum = 0.f;
+    if (vec) {
+#pragma unroll
+        for (int c = 0; c < kKeep; ++c) {
+            const int i = threadIdx.x + c * kThreads;
+            if (i < chunks) {
+                keep[c] = reinterpret_cast<const float4*>(xr)[i];
+                sum += (keep[c].x * keep[c].x + keep[c].y * keep[c].y) + (keep[c].z * keep[c].z + keep[c].w * keep[c].w);
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < size; i += kThreads) sum = fmaf(xr[i], xr[i], sum);
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = sum;
+    __syncthreads();
+    sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kThreads / 32; ++i) sum += part[i];
+    const float scale = 1.0f / sqrtf(sum / static_cast<float>(size) + eps);
+    if (vec) {
+#pragma unroll
+        for (int c = 0; c < kKeep; ++c) {
+            const int i = threadIdx.x + c * kThreads;
+            if (i < chunks) {
+                const float4 wv = reinterpret_cast<const float4*>(w)[i];
+                float4 v = keep[c];
+                v.x *= scale * (wv.x + w_offset), v.y *= scale * (wv.y + w_offset);
+                v.z *= scale * (wv.z + w_offset), v.w *= scale * (wv.w + w_offset);
+                store4(yr + 4 * i, v);
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < size; i += kThreads) yr[i] = Elt<T>::from_float(xr[i] * scale * (w[i] + w_offset));
+    }
+}
+
+}  // namespace
+}  // namespace b2kv
+
+using namespace b2kv;
+
+extern "C" int b2kv_embed_rows(const void* table, const int32_t* ids, float* out, int rows, int dim, int vocab, int dtype,
+                               int32_t* dev_status, void* stream) {
+    if (elt_bytes(dtype) == 0) return B2KV_ERR_UNSUPPORTED;
+    if (!table || !ids || !out || rows <= 0 || dim <= 0 || vocab <= 0) return B2KV_ERR_BAD_ARG;
+    OverlapLaunch launch(rows, kThreads, 0, stream);
+    if (dtype == B2KV_DTYPE_F32)
+        B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, embed_rows_kernel<float>, static_cast<const float*>(table), ids, out, dim,
+                                         vocab, dev_status));
+    else
+        B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, embed_rows_kernel<__nv_bfloat16>, static_cast<const __nv_bfloat16*>(table),
+                                         ids, out, dim, vocab, dev_status));
+    return B2KV_OK;
+}
+
+extern "C" int b2kv_rmsnorm(const float* x, int64_t ld_x, const int32_t* row_index, const float* w, float w_offset, void* out,
+                            int64_t ld_out, int rows, int size, float eps, int dtype, void* stream) {
+    if (elt_bytes(dtype) == 0) return B2KV_ERR_UNSUPPORTED;
+    if (!x || !w || !out || rows <= 0 || size <= 0 || ld_x < size || ld_out < size) return B2KV_ERR_BAD_ARG;
+    const bool vec = size % 4 == 0 && ld_x % 4 == 0 && ld_out % 4 == 0 && size <= 16384 && aligned16(x) && aligned16(w) && aligned16(out);
+    OverlapLaunch launch(rows, kThreads, 0, stream);
+    if (dtype == B2KV_DTYPE_F32)
+        B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, rmsnorm_kernel<float>, x, ld_x, row_index, w, w_offset,
+                                         static_cast<float*>(out), ld_out, size, eps, vec));
+    else
+        B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, rmsnorm_kernel<__nv_bfloat16>, x, ld_x, row_index, w, w_offset,
+                                         static_cast<__nv_bfloat16*>(out), ld_out, size, eps, vec));
+    return B2KV_OK;
+}

@@ -61,6 +61,8 @@ def kv_cache_create(ctx: GPUContext, config: KVCacheConfig) -> KVCache:
     if config.layout not in ("bthd", "bhtd"):
         raise ValueError(f"layout must be 'bthd' or 'bhtd', got {config.layout!r}")
     dtype_code(config.dtype)
+    if config.v_head_dim < 0 or (config.v_head_dim > 0 and config.block_size > 0):
+        raise ValueError("v_head_dim must be >= 0, and a paged cache has K and V rows of one width")
 
     B, T, H, D = config.batch_size, config.max_seq_len, config.n_heads, config.head_dim
     paged = config.block_size > 0
@@ -82,7 +84,7 @@ def kv_cache_create(ctx: GPUContext, config: KVCacheConfig) -> KVCache:
     layers: List[KVCacheLayer] = []
     for _ in range(config.n_layers):
         k_cache = gpu_buffer_2d_create(ctx, rows, cols, dtype=config.dtype)
-        v_cache = gpu_buffer_2d_create(ctx, rows, cols, dtype=config.dtype)
+        v_cache = gpu_buffer_2d_create(ctx, rows, cols // D * (config.v_head_dim or D), dtype=config.dtype)
         gpu_buffer_zerofy(ctx, k_cache)
         gpu_buffer_zerofy(ctx, v_cache)
         layers.append(KVCacheLayer(k_cache=k_cache, v_cache=v_cache))
@@ -90,7 +92,7 @@ def kv_cache_create(ctx: GPUContext, config: KVCacheConfig) -> KVCache:
     seq_lens = torch.zeros(B, dtype=torch.int32, device=ctx.device) if config.ragged else None
     return KVCache(layers=layers, batch_size=B, max_seq_len=T, current_len=0, n_heads=H, head_dim=D,
                    dtype=config.dtype, layout=config.layout, seq_lens=seq_lens, block_table=block_table,
-                   block_size=config.block_size if paged else 0, n_blocks=n_blocks)
+                   block_size=config.block_size if paged else 0, n_blocks=n_blocks, v_head_dim=config.v_head_dim)
 
 
 def kv_cache_reset(cache: KVCache) -> None:
@@ -112,6 +114,11 @@ def kv_cache_set_lengths(cache: KVCache, lens) -> None:
     cache.current_len = int(host.max())
 
 
+def _same_width(cache: KVCache) -> None:
+    if cache.v_head_dim not in (0, cache.head_dim):
+        raise ValueError("a latent cache (v_head_dim set) is filled and read by the latent attention operations")
+
+
 def _ptr(t: Optional[torch.Tensor]) -> Optional[int]:
     return None if t is None else t.data_ptr()
 
@@ -123,6 +130,7 @@ def kv_cache_update(ctx: GPUContext, cache: KVCache, layer_idx: int, new_k: GPUB
         raise ValueError(f"layer_idx {layer_idx} out of range [0, {len(cache.layers)})")
     if cache.current_len >= cache.max_seq_len:
         raise ValueError(f"Cache is full: current_len={cache.current_len}, max_seq_len={cache.max_seq_len}")
+    _same_width(cache)
     embedding_dim = cache.n_heads * cache.head_dim
     expected_rows = cache.batch_size * 1
     validate_buffer_shape_2d(new_k, (expected_rows, embedding_dim), "new_k")
@@ -177,6 +185,7 @@ def attention_with_kv_cache(ctx: GPUContext, cache: KVCache, layer_idx: int, q_n
                 f"sequence length ({workgroup_size}) for attention_with_kv_cache. "
                 f"Use chunked attention or increase workgroup_size in config."
             )
+    _same_width(cache)
     embedding_dim = cache.n_heads * cache.head_dim
     expected_q_rows = cache.batch_size * 1
     validate_buffer_shape_2d(q_new, (expected_q_rows, embedding_dim), "q_new")
@@ -214,19 +223,19 @@ def kv_cache_gather(ctx: GPUContext, cache: KVCache, layer_idx: int, which: str 
     T_out = cache.max_seq_len if length is None else int(length)
     layer = cache.layers[layer_idx]
     src = layer.k_cache if which == "k" else layer.v_cache
-    out = torch.empty((cache.batch_size, T_out, cache.n_heads, cache.head_dim), dtype=cache.dtype,
-                      device=src.buffer.device)
+    D = cache.head_dim if which == "k" else (cache.v_head_dim or cache.head_dim)
+    out = torch.empty((cache.batch_size, T_out, cache.n_heads, D), dtype=cache.dtype, device=src.buffer.device)
     stream = batch_op_begin(ctx)
-    s0, st, sh = cache_strides(cache)
+    s0, st, sh = (s // cache.head_dim * D for s in cache_strides(cache))
     dt = dtype_code(cache.dtype)
     n = min(cache.current_len, T_out)
     if cache.block_table is None:
         rc = _native.lib.b2kv_gather(src.buffer.data_ptr(), out.data_ptr(), _ptr(cache.seq_lens), n,
-                                     cache.batch_size, cache.n_heads, cache.head_dim, T_out, s0, st, sh, dt, stream)
+                                     cache.batch_size, cache.n_heads, D, T_out, s0, st, sh, dt, stream)
     else:
         rc = _native.lib.b2kv_gather_paged(src.buffer.data_ptr(), out.data_ptr(), _ptr(cache.seq_lens), n,
                                            cache.block_table.data_ptr(), cache.block_table.shape[1], cache.block_size,
-                                           cache.n_blocks, cache.batch_size, cache.n_heads, cache.head_dim, T_out,
+                                           cache.n_blocks, cache.batch_size, cache.n_heads, D, T_out,
                                            s0, st, sh, dt, dev_status_ptr(ctx), stream)
     _native.check(rc)
     return out

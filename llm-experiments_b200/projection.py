@@ -10,9 +10,14 @@ the cache.  Checks and texts follow ``kv_cache_update``; bf16 caches with a cont
 """
 from __future__ import annotations
 
+import ctypes
+from dataclasses import dataclass
+from typing import Optional, Sequence
+
 import torch
 
 from . import _native
+from ._native import SEG_F32, SEG_GLU_CLAMP, SEG_GLU_SILU, SEG_STORE  # noqa: F401
 from .batch import batch_op_begin, dev_status_ptr, reference_op, validate_buffer_shape_2d
 from .kv_cache import _ptr, cache_strides, dtype_code
 from .types import GPUBuffer2D, GPUContext, KVCache
@@ -97,3 +102,54 @@ def qkv_project_append(ctx: GPUContext, cache: KVCache, layer_idx: int, x: GPUBu
             # stream-ordered after the kernel, which read the old positions
             _native.check(_native.lib.b2kv_advance_lengths(cache.seq_lens.data_ptr(), cache.batch_size, 1, stream))
         cache.current_len += 1
+
+
+@dataclass
+class OutputSegment:
+    """Columns of a linear layer's weight up to ``end`` (from the end of the segment before) and where their products go:
+    ``SEG_STORE`` in the storage type, ``SEG_F32`` in fp32 (with the residual added), ``SEG_GLU_SILU`` / ``SEG_GLU_CLAMP``
+    as gated pairs, (gate, up) in neighbouring columns, giving half as many output columns.  ``out`` may be a view of some
+    columns of a wider buffer; group g of a grouped product writes ``group`` elements further on per group."""
+
+    end: int
+    kind: int
+    out: GPUBuffer2D
+    group: int = 0
+
+
+@reference_op("linear")
+def linear(ctx: GPUContext, x: GPUBuffer2D, w: GPUBuffer2D, k: int, segments: Sequence[OutputSegment],
+           residual: Optional[GPUBuffer2D] = None, limit: float = 0.0, groups: int = 1, group_x: int = 0, group_w: int = 0,
+           group_rows: Optional[torch.Tensor] = None, max_group_rows: int = 0, path: int = 0) -> None:
+    """``x @ w`` with the output columns cut into segments, fp32 or bfloat16 storage, any sizes (``b2kv_linear``).
+
+    ``x`` ``[rows, >= k]`` and ``w`` (rows of the weight matrix, ``[in, out]``) may be views with a row pitch.  With
+    ``groups`` > 1, group g reads ``x`` from element ``g * group_x`` on and ``w`` from ``g * group_w`` on (the heads of a
+    per-head product), or, with ``group_rows`` (int32 ``[groups + 1]`` on the device), rows ``group_rows[g] ..
+    group_rows[g + 1] - 1`` of ``x`` (the experts of a mixture; at most ``max_group_rows`` rows each).  ``path`` forces a
+    kernel (1 CUDA cores, 2 weight streaming, 3 tiled)."""
+    rows, n = x.shape[0], segments[-1].end
+    if rows <= 0 or k <= 0 or n <= 0:
+        raise ValueError(f"linear: Invalid dimensions x=({rows}, {k}), w=({k}, {n})")
+    if x.buffer.dtype != w.buffer.dtype or any(t.buffer.stride(1) != 1 for t in (x, w)):
+        raise ValueError("linear: x and w must share one dtype and have contiguous rows")
+    if w.shape[1] < n or (group_x == 0 and x.shape[1] < k):
+        raise ValueError(f"linear: Dimension mismatch x {tuple(x.shape)}, w {tuple(w.shape)}, k={k}, n={n}")
+    a = _native.LinearArgs(x=x.buffer.data_ptr(), w=w.buffer.data_ptr(), ld_x=x.buffer.stride(0), group_x=group_x,
+                           ld_w=w.buffer.stride(0), group_w=group_w, rows=rows, K=k, N=n, groups=groups,
+                           max_group_rows=max_group_rows, n_seg=len(segments), dtype=dtype_code(x.buffer.dtype), path=path,
+                           limit=limit)
+    for i, s in enumerate(segments):
+        want = torch.float32 if s.kind == SEG_F32 else x.buffer.dtype
+        if s.out.buffer.dtype != want or s.out.buffer.stride(1) != 1 or s.out.shape[0] < rows:
+            raise ValueError(f"linear: output of segment {i} must be {want} with at least {rows} rows of contiguous elements")
+        a.seg[i] = _native.Segment(out=s.out.buffer.data_ptr(), ld=s.out.buffer.stride(0), group=s.group, end=s.end,
+                                   kind=s.kind)
+    if residual is not None:
+        if residual.buffer.dtype != torch.float32:
+            raise ValueError("linear: the residual must be float32")
+        a.residual, a.ld_residual = residual.buffer.data_ptr(), residual.buffer.stride(0)
+    if group_rows is not None:
+        a.group_rows = group_rows.data_ptr()
+    stream = batch_op_begin(ctx)
+    _native.check(_native.lib.b2kv_linear(ctypes.byref(a), dev_status_ptr(ctx), stream))

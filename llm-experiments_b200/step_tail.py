@@ -92,6 +92,33 @@ def layernorm(ctx: GPUContext, input_buf: GPUBuffer2D, gamma: GPUBuffer1D, beta:
     _native.check(fn(*ptrs, n_elements, size, float(ctx.config.layernorm_epsilon), stream))
 
 
+@reference_op("embedding")
+def embedding_rows(ctx: GPUContext, table: GPUBuffer2D, ids: torch.Tensor, output: GPUBuffer2D) -> None:
+    """``output[i] = table[ids[i]]`` as fp32 rows, no position added: the start of a 32-bit residual stream."""
+    rows, dim = output.shape
+    if table.shape[1] != dim or ids.numel() < rows or ids.dtype != torch.int32:
+        raise ValueError("embedding_rows needs one int32 id per output row and a table of the output's width")
+    stream = batch_op_begin(ctx)
+    _native.check(_native.lib.b2kv_embed_rows(table.buffer.data_ptr(), ids.data_ptr(), _f32(output, "output"), rows, dim,
+                                              table.shape[0], _DTYPE_CODES[table.buffer.dtype], dev_status_ptr(ctx), stream))
+
+
+@reference_op("rms_norm")
+def rms_norm(ctx: GPUContext, x: GPUBuffer2D, weight: GPUBuffer1D, output: GPUBuffer2D, eps: float,
+             weight_offset: float = 0.0, row_index: torch.Tensor = None) -> None:
+    """``output[i] = x[r] / sqrt(mean(x[r]^2) + eps) * (weight + weight_offset)`` with ``r = row_index[i]`` (or ``i``); fp32
+    rows in, float32 or bfloat16 rows out.  ``weight_offset=1`` is the norm whose weight is stored around zero."""
+    rows, size = output.shape
+    validate_buffer_shape_1d(weight, size, "weight")
+    if x.shape[1] != size or (row_index is None and x.shape[0] < rows):
+        raise ValueError(f"rms_norm shape mismatch: x {tuple(x.shape)}, output {tuple(output.shape)}")
+    stream = batch_op_begin(ctx)
+    _native.check(_native.lib.b2kv_rmsnorm(_f32(x, "x"), x.buffer.stride(0),
+                                           None if row_index is None else row_index.data_ptr(), _f32(weight, "weight"),
+                                           weight_offset, output.buffer.data_ptr(), output.buffer.stride(0), rows, size, eps,
+                                           _DTYPE_CODES[output.buffer.dtype], stream))
+
+
 @reference_op("extract_last_tokens")
 def extract_last_tokens(ctx: GPUContext, input_buf: GPUBuffer2D, output: GPUBuffer2D, batch_size: int, seq_len: int,
                         embedding_dim: int) -> None:

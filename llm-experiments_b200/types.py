@@ -121,7 +121,9 @@ class GPUContext:
 @dataclass
 class KVCacheLayer:
     """K and V of one layer.  Reference layout (default): ``[B*T_max, H*D]``.
-    ``layout="bhtd"``: ``[B*H*T_max, D]``.  Paged: pools ``[n_blocks*H*block_size, D]``."""
+    ``layout="bhtd"``: ``[B*H*T_max, D]``.  Paged: pools ``[n_blocks*H*block_size, D]``.
+    A latent layer (``v_head_dim`` set, one head) keeps the rotated key part in ``k_cache`` and the latent row, from which
+    its heads' keys and values are made, in ``v_cache``."""
 
     k_cache: GPUBuffer2D
     v_cache: GPUBuffer2D
@@ -143,6 +145,7 @@ class KVCache:
     block_size: int = 0
     n_blocks: int = 0
     workspace: Optional[torch.Tensor] = None  # decode scratch, allocated on first use
+    v_head_dim: int = 0  # row width of V where it differs from K's head_dim (latent layers); 0 = head_dim
 
 
 @dataclass
@@ -158,3 +161,4 @@ class KVCacheConfig:
     ragged: bool = False  # keep per-sequence lengths on the device
     block_size: int = 0  # > 0: paged cache with blocks of this many tokens
     n_blocks: int = 0  # pool size in blocks (paged)
+    v_head_dim: int = 0  # > 0: V rows are this wide (latent layers; contiguous caches only)
