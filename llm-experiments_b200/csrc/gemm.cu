@@ -23,8 +23,14 @@
 // port.  Rows, columns and input features past the matrix edges are zero-filled by the tensor maps and masked
 // in the epilogue.  Every mbarrier wait is bounded; a wait that runs out makes all warps leave through the
 // common exit, where the tensor memory is released.
+//
+// b2kv_linear's products of many rows run on the same two kernels with another kind of parameters (SegParams below): output
+// columns cut into segments with places and forms of their own (bf16, fp32 with residual, gated pairs), and optionally rows
+// grouped by expert, each group with a weight matrix of its own; the tiles of all groups then form one list, whose length is
+// read from the device.
 #include <algorithm>
 
+#include "linear.cuh"
 #include "tc_ptx.cuh"
 #include "tma_map.cuh"
 
@@ -55,6 +61,29 @@ struct GemmParams {
     int32_t* dev_status;  // optional status word: receives B2KV_DEV_WAIT_TIMEOUT when a bounded wait ran out
 };
 
+// b2kv_linear: segments and, with group_rows, groups of rows.
+constexpr int kMaxGroups = 1024;
+struct SegParams {
+    b2kv_linear_args a;
+    int M, N, K;
+    int tiles_m, tiles_n;
+    int32_t* dev_status;
+};
+
+// Output tile: first row of A, row behind the last one that belongs to the tile's group, column tile, first row of W.
+struct Tile {
+    int row0, row_end, tn, k_row0;
+};
+
+// First row tile of every group (and behind the last one), for tiles of tile_rows rows; in shared memory, empty for
+// parameters without groups.
+template <typename P>
+struct GroupTable {};
+template <>
+struct GroupTable<SegParams> {
+    int first[kMaxGroups + 1];
+};
+
 struct SharedStorage {
     alignas(1024) uint8_t stage[kStages][kStageBytes];
     alignas(8) uint64_t full[kStages];
@@ -73,7 +102,8 @@ __device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* map, u
 
 // Tile t of the order described above -> (row tile, column tile): column bands outermost, then row bands,
 // then the tiles of a block with the row tile running fastest.
-__device__ __forceinline__ void tile_coords(int t, const GemmParams& p, int& tm, int& tn) {
+template <typename P>
+__device__ __forceinline__ void tile_coords(int t, const P& p, int& tm, int& tn) {
     const int cband_tiles = p.tiles_m * kBandCols;
     const int cband = t / cband_tiles;  // only the last column band can be narrower, and nothing follows it
     const int first_col = cband * kBandCols;
@@ -88,14 +118,63 @@ __device__ __forceinline__ void tile_coords(int t, const GemmParams& p, int& tm,
     tn = first_col + within / rows_here;
 }
 
-__device__ __forceinline__ void epilogue_rows(const GemmParams& p, uint32_t t_addr, int grow, int col_base);
+// Set up by the whole CTA before the roles part; returns the number of output tiles.
+__device__ __forceinline__ int setup_tiles(const GemmParams& p, GroupTable<GemmParams>&, int) { return p.tiles_m * p.tiles_n; }
+__device__ __forceinline__ int setup_tiles(const SegParams& p, GroupTable<SegParams>& table, int tile_rows) {
+    if (p.a.group_rows == nullptr) return p.tiles_m * p.tiles_n;
+    if (threadIdx.x < 32) {  // one warp scans the groups' tile counts, 32 groups at a time
+        int base = 0;
+        for (int g0 = 0; g0 < p.a.groups; g0 += 32) {
+            const int g = g0 + static_cast<int>(threadIdx.x);
+            int n = g < p.a.groups ? (p.a.group_rows[g + 1] - p.a.group_rows[g] + tile_rows - 1) / tile_rows : 0;
+#pragma unroll
+            for (int off = 1; off < 32; off <<= 1) {
+                const int up = __shfl_up_sync(0xffffffffu, n, off);
+                if (static_cast<int>(threadIdx.x) >= off) n += up;
+            }
+            if (g < p.a.groups) table.first[g + 1] = base + n;
+            base += __shfl_sync(0xffffffffu, n, 31);
+        }
+        if (threadIdx.x == 0) table.first[0] = 0;
+    }
+    __syncthreads();
+    return table.first[p.a.groups] * p.tiles_n;
+}
 
+__device__ __forceinline__ Tile find_tile(int t, const GemmParams& p, const GroupTable<GemmParams>&, int tile_rows) {
+    int tm, tn;
+    tile_coords(t, p, tm, tn);
+    return {tm * tile_rows, p.M, tn, 0};
+}
+__device__ __forceinline__ Tile find_tile(int t, const SegParams& p, const GroupTable<SegParams>& table, int tile_rows) {
+    if (p.a.group_rows == nullptr) {
+        int tm, tn;
+        tile_coords(t, p, tm, tn);
+        return {tm * tile_rows, p.M, tn, 0};
+    }
+    int lo = 0, hi = p.a.groups - 1;  // the last group whose first tile is not behind t (so it has tiles)
+    while (lo < hi) {
+        const int mid = (lo + hi + 1) / 2;
+        if (table.first[mid] * p.tiles_n <= t) lo = mid;
+        else hi = mid - 1;
+    }
+    const int first = table.first[lo], rows_here = table.first[lo + 1] - first;
+    const int within = t - first * p.tiles_n;  // row tiles run fastest: they share the group's columns of W
+    return {p.a.group_rows[lo] + within % rows_here * tile_rows, p.a.group_rows[lo + 1], within / rows_here, lo * p.K};
+}
+
+__device__ __forceinline__ void epilogue_rows(const GemmParams& p, uint32_t t_addr, int grow, int row_end, int col_base);
+__device__ __forceinline__ void epilogue_rows(const SegParams& p, uint32_t t_addr, int grow, int row_end, int col_base);
+
+template <typename P>
 __global__ void __launch_bounds__(kThreads, 1)
-gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__ CUtensorMap tm_w, const GemmParams p) {
+gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__ CUtensorMap tm_w,
+               const __grid_constant__ P p) {
+    __shared__ GroupTable<P> table;
     extern __shared__ uint8_t smem_raw[];
     SharedStorage& sm = *reinterpret_cast<SharedStorage*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int n_tiles = p.tiles_m * p.tiles_n;
+    const int n_tiles = setup_tiles(p, table, kBM);
     const int n_k = (p.K + kBK - 1) / kBK;
 
     if (threadIdx.x == 0) {
@@ -125,17 +204,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
             bool ok = true;
             uint32_t it = 0;  // stages filled so far: stage it % kStages, phase it / kStages
             for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x) {
-                int tm, tn;
-                tile_coords(t, p, tm, tn);
+                const Tile tl = find_tile(t, p, table, kBM);
                 for (int kb = 0; kb < n_k; ++kb, ++it) {
                     const int s = it % kStages;
                     ok = mbar_wait(&sm.empty[s], ((it / kStages) & 1) ^ 1);
                     if (!ok) break;
                     mbar_arrive_expect_tx(&sm.full[s], kStageBytes);
-                    tma_load_2d(sm.stage[s], &tm_a, &sm.full[s], kb * kBK, tm * kBM);
+                    tma_load_2d(sm.stage[s], &tm_a, &sm.full[s], kb * kBK, tl.row0);
 #pragma unroll
                     for (int sp = 0; sp < kBN / 64; ++sp)
-                        tma_load_2d(sm.stage[s] + kABytes + sp * kWSpanBytes, &tm_w, &sm.full[s], tn * kBN + sp * 64, kb * kBK);
+                        tma_load_2d(sm.stage[s] + kABytes + sp * kWSpanBytes, &tm_w, &sm.full[s], tl.tn * kBN + sp * 64,
+                                    tl.k_row0 + kb * kBK);
                 }
             }
             if (!ok) sm.abort_flag = 1;
@@ -182,13 +261,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__
         bool ok = true;
         uint32_t local = 0;
         for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x, ++local) {
-            int tm, tn;
-            tile_coords(t, p, tm, tn);
+            const Tile tl = find_tile(t, p, table, kBM);
             const uint32_t buf = local & 1;
             ok = mbar_wait(&sm.acc_full[buf], (local >> 1) & 1);
             if (!ok) break;
             tc_fence_after();
-            epilogue_rows(p, tmem + lane_base + buf * kBN, tm * kBM + row, tn * kBN);
+            epilogue_rows(p, tmem + lane_base + buf * kBN, tl.row0 + row, tl.row_end, tl.tn * kBN);
             // this warp has read its lanes of the accumulator: hand it back to the MMA issuer
             tc_fence_before();
             __syncwarp();
@@ -292,9 +370,9 @@ __device__ __forceinline__ void mma_ss_pair(uint32_t d_tmem, uint64_t a_desc, ui
         : "memory");
 }
 
-// Epilogue of one accumulator for one warp: thread = output row `grow` (TMEM lane of `t_addr`), columns
-// [col_base, col_base + 256) clipped to N.
-__device__ __forceinline__ void epilogue_rows(const GemmParams& p, uint32_t t_addr, int grow, int col_base) {
+// Epilogue of one accumulator for one warp: thread = output row `grow` (TMEM lane of `t_addr`; rows from row_end on are
+// not stored), columns [col_base, col_base + 256) clipped to N.
+__device__ __forceinline__ void epilogue_rows(const GemmParams& p, uint32_t t_addr, int grow, int row_end, int col_base) {
     const size_t row_off = static_cast<size_t>(grow) * p.N;
 #pragma unroll 1
     for (int c = 0; c < kBN / 32; ++c) {
@@ -303,7 +381,7 @@ __device__ __forceinline__ void epilogue_rows(const GemmParams& p, uint32_t t_ad
         uint32_t acc[32];
         tmem_ld32(t_addr + c * 32, acc);
         tmem_wait_ld();
-        if (grow < p.M) {
+        if (grow < row_end) {
 #pragma unroll
             for (int v = 0; v < 4; ++v) {
                 const int col = col0 + v * 8;
@@ -344,9 +422,74 @@ __device__ __forceinline__ void epilogue_rows(const GemmParams& p, uint32_t t_ad
     }
 }
 
-template <int kBKP, int kStagesP>
+// The same for segments (32 columns never straddle a boundary).
+__device__ __forceinline__ void epilogue_rows(const SegParams& p, uint32_t t_addr, int grow, int row_end, int col_base) {
+    const bool live = grow < row_end;
+#pragma unroll 1
+    for (int c = 0; c < kBN / 32; ++c) {
+        const int col0 = col_base + c * 32;
+        if (col0 >= p.N) break;
+        uint32_t acc[32];
+        tmem_ld32(t_addr + c * 32, acc);
+        const int s = lin::segment_of(p.a, col0);
+        const b2kv_segment& sg = p.a.seg[s];
+        const int local = col0 - lin::segment_first(p.a, s);
+        tmem_wait_ld();
+        if (!live) continue;
+        const int64_t row = grow;
+        if (sg.kind == B2KV_SEG_F32) {
+            float* out = static_cast<float*>(sg.out) + row * sg.ld + local;
+            const float* res = p.a.residual ? p.a.residual + row * p.a.ld_residual + local : nullptr;
+            float4 add[8];
+#pragma unroll
+            for (int v = 0; v < 8; ++v)
+                add[v] = (res != nullptr && col0 + v * 4 < p.N) ? *reinterpret_cast<const float4*>(res + v * 4)
+                                                                : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int v = 0; v < 8; ++v) {
+                if (col0 + v * 4 >= p.N) break;
+                float4 o;
+                o.x = __uint_as_float(acc[v * 4 + 0]) + add[v].x, o.y = __uint_as_float(acc[v * 4 + 1]) + add[v].y;
+                o.z = __uint_as_float(acc[v * 4 + 2]) + add[v].z, o.w = __uint_as_float(acc[v * 4 + 3]) + add[v].w;
+                *reinterpret_cast<float4*>(out + v * 4) = o;
+            }
+        } else if (sg.kind == B2KV_SEG_STORE) {
+            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(sg.out) + row * sg.ld + local;
+#pragma unroll
+            for (int v = 0; v < 4; ++v) {
+                if (col0 + v * 8 >= p.N) break;
+                uint4 w;
+                w.x = pack_bf16(__uint_as_float(acc[v * 8 + 0]), __uint_as_float(acc[v * 8 + 1]));
+                w.y = pack_bf16(__uint_as_float(acc[v * 8 + 2]), __uint_as_float(acc[v * 8 + 3]));
+                w.z = pack_bf16(__uint_as_float(acc[v * 8 + 4]), __uint_as_float(acc[v * 8 + 5]));
+                w.w = pack_bf16(__uint_as_float(acc[v * 8 + 6]), __uint_as_float(acc[v * 8 + 7]));
+                *reinterpret_cast<uint4*>(out + v * 8) = w;
+            }
+        } else {
+            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(sg.out) + row * sg.ld + local / 2;
+            float z[16];
+#pragma unroll
+            for (int i = 0; i < 16; ++i)
+                z[i] = lin::glu(sg.kind, __uint_as_float(acc[2 * i]), __uint_as_float(acc[2 * i + 1]), p.a.limit);
+#pragma unroll
+            for (int v = 0; v < 2; ++v) {
+                if (col0 + v * 16 >= p.N) break;
+                uint4 w;
+                w.x = pack_bf16(z[v * 8 + 0], z[v * 8 + 1]);
+                w.y = pack_bf16(z[v * 8 + 2], z[v * 8 + 3]);
+                w.z = pack_bf16(z[v * 8 + 4], z[v * 8 + 5]);
+                w.w = pack_bf16(z[v * 8 + 6], z[v * 8 + 7]);
+                *reinterpret_cast<uint4*>(out + v * 8) = w;
+            }
+        }
+    }
+}
+
+template <int kBKP, int kStagesP, typename P>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads, 1)
-gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__ CUtensorMap tm_w, const GemmParams p) {
+gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__ CUtensorMap tm_w,
+                 const __grid_constant__ P p) {
+    __shared__ GroupTable<P> table;
     extern __shared__ uint8_t smem_raw[];
     using Smem = PairStorage<kBKP, kStagesP>;
     constexpr int kABytesP = Smem::kABytesP, kWSpanP = Smem::kWSpanP, kStageBytesP = Smem::kStageBytesP;
@@ -354,7 +497,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r = static_cast<int>(cluster_ctarank());  // 0 = leader
     const int cid = blockIdx.x >> 1, n_clusters = gridDim.x >> 1;
-    const int n_tiles = p.tiles_m * p.tiles_n;  // tiles of 256 rows x 256 columns
+    const int n_tiles = setup_tiles(p, table, 2 * kBM);  // tiles of 256 rows x 256 columns
     const int n_k = (p.K + kBKP - 1) / kBKP;
 
     if (threadIdx.x == 0) {
@@ -385,8 +528,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
             bool ok = true;
             uint32_t it = 0;
             for (int t = cid; t < n_tiles && ok; t += n_clusters) {
-                int tm, tn;
-                tile_coords(t, p, tm, tn);
+                const Tile tl = find_tile(t, p, table, 2 * kBM);
                 for (int kb = 0; kb < n_k; ++kb, ++it) {
                     const int s = it % kStagesP;
                     ok = mbar_wait(&sm.empty[s], ((it / kStagesP) & 1) ^ 1);
@@ -396,11 +538,11 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
 #pragma unroll
                     for (int ks = 0; ks < kBKP / 64; ++ks)  // 64 input features (one swizzle span) per box of A
                         tma_load_2d_pair(sm.stage[s] + ks * (kBM * 128), &tm_a, lead_full, kb * kBKP + ks * 64,
-                                         tm * 2 * kBM + r * kBM);
+                                         tl.row0 + r * kBM);
 #pragma unroll
                     for (int sp = 0; sp < 2; ++sp)
                         tma_load_2d_pair(sm.stage[s] + kABytesP + sp * kWSpanP, &tm_w, lead_full,
-                                         tn * kBN + r * (kBN / 2) + sp * 64, kb * kBKP);
+                                         tl.tn * kBN + r * (kBN / 2) + sp * 64, tl.k_row0 + kb * kBKP);
                 }
             }
             if (!ok) sm.abort_flag = 1;
@@ -447,13 +589,12 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
         bool ok = true;
         uint32_t local = 0;
         for (int t = cid; t < n_tiles && ok; t += n_clusters, ++local) {
-            int tm, tn;
-            tile_coords(t, p, tm, tn);
+            const Tile tl = find_tile(t, p, table, 2 * kBM);
             const uint32_t buf = local & 1;
             ok = mbar_wait(&sm.acc_full[buf], (local >> 1) & 1);
             if (!ok) break;
             tc_fence_after();
-            epilogue_rows(p, tmem + lane_base + buf * kBN, tm * 2 * kBM + r * kBM + row, tn * kBN);
+            epilogue_rows(p, tmem + lane_base + buf * kBN, tl.row0 + r * kBM + row, tl.row_end, tl.tn * kBN);
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive_cluster(map_to_cta(&sm.acc_empty[buf], 0));
@@ -475,11 +616,11 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant
 
 // [rows, cols] bf16 row-major matrix, boxes of box_rows x 64 columns, 128-byte swizzle; reads outside the
 // matrix give zero.
-static bool make_map(CUtensorMap* map, const void* base, int rows, int cols, int box_rows) {
+static bool make_map(CUtensorMap* map, const void* base, int64_t rows, int cols, int64_t pitch, int box_rows) {
     EncodeTiledFn fn = tensor_map_encoder();
     if (fn == nullptr) return false;
     const cuuint64_t dims[2] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(rows)};
-    const cuuint64_t strides[1] = {static_cast<cuuint64_t>(cols) * 2};
+    const cuuint64_t strides[1] = {static_cast<cuuint64_t>(pitch) * 2};
     const cuuint32_t box[2] = {64, static_cast<cuuint32_t>(box_rows)};
     const cuuint32_t estr[2] = {1, 1};
     return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
@@ -487,35 +628,24 @@ static bool make_map(CUtensorMap* map, const void* base, int rows, int cols, int
               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-}  // namespace gemm
-
-}  // namespace b2kv
-
-using namespace b2kv;
-
-extern "C" int b2kv_matmul(const void* a, const void* w, const void* bias, const void* residual, void* out, int M, int K,
-                           int N, int activation, int dtype, int32_t* dev_status, void* stream) {
-    if (dtype != B2KV_DTYPE_BF16) return B2KV_ERR_UNSUPPORTED;
-    if (!a || !w || !out) return B2KV_ERR_BAD_ARG;
-    if (M <= 0 || K <= 0 || N <= 0 || activation < 0 || activation > 1) return B2KV_ERR_BAD_ARG;
-    // row pitches must be multiples of 16 bytes (tensor maps, 16-byte epilogue accesses)
-    if (K % 8 != 0 || N % 8 != 0) return B2KV_ERR_UNSUPPORTED;
-    if (!aligned16(a) || !aligned16(w) || !aligned16(out) || !aligned16(residual) || !aligned16(bias)) return B2KV_ERR_ALIGN;
-    const long long tiles_m = (static_cast<long long>(M) + gemm::kBM - 1) / gemm::kBM;
-    const long long tiles_n = (static_cast<long long>(N) + gemm::kBN - 1) / gemm::kBN;
-    if (tiles_m * tiles_n > 0x3fffffffLL) return B2KV_ERR_UNSUPPORTED;
+// Chooses the form and launches it.  max_tiles_m: row tiles of kBM rows at most; tall: whether 256-row tiles pay.
+template <typename P>
+static int launch(P p, const void* a, int64_t a_rows, int64_t lda, const void* w, int64_t w_rows, int64_t ldw, long long max_tiles_m,
+                  long long max_tiles_m_pair, bool tall, void* stream) {
+    const long long tiles_n = (static_cast<long long>(p.N) + kBN - 1) / kBN;
+    if (max_tiles_m * tiles_n > 0x3fffffffLL) return B2KV_ERR_UNSUPPORTED;
     CUtensorMap ta, tw;
-    if (!gemm::make_map(&ta, a, M, K, gemm::kBM) || !gemm::make_map(&tw, w, K, N, gemm::kBK)) return B2KV_ERR_UNSUPPORTED;
-    gemm::GemmParams p{static_cast<const __nv_bfloat16*>(bias), static_cast<const __nv_bfloat16*>(residual),
-                       static_cast<__nv_bfloat16*>(out), M, N, K, activation, static_cast<int>(tiles_m),
-                       static_cast<int>(tiles_n), dev_status};
-    constexpr size_t smem = sizeof(gemm::SharedStorage) + 1024;
-    using Pair64 = gemm::PairStorage<64, 6>;
-    using Pair128 = gemm::PairStorage<128, 3>;
+    if (!make_map(&ta, a, a_rows, p.K, lda, kBM) || !make_map(&tw, w, w_rows, p.N, ldw, kBK)) return B2KV_ERR_UNSUPPORTED;
+    p.tiles_m = static_cast<int>(max_tiles_m);
+    p.tiles_n = static_cast<int>(tiles_n);
+    constexpr size_t smem = sizeof(SharedStorage) + 1024;
+    using Pair64 = PairStorage<64, 6>;
+    using Pair128 = PairStorage<128, 3>;
     constexpr size_t smem_pair = sizeof(Pair64) + 1024;
     constexpr size_t smem_pair128 = sizeof(Pair128) + 1024;
-    auto pair64 = gemm::gemm_pair_kernel<64, 6>;
-    auto pair128 = gemm::gemm_pair_kernel<128, 3>;
+    auto single = gemm_tc_kernel<P>;
+    auto pair64 = gemm_pair_kernel<64, 6, P>;
+    auto pair128 = gemm_pair_kernel<128, 3, P>;
     static bool configured[64] = {false};
     static int sm_count[64] = {0};
     static int max_clusters[64] = {0};  // CTA pairs of gemm_pair_kernel that can be resident together
@@ -525,7 +655,7 @@ extern "C" int b2kv_matmul(const void* a, const void* w, const void* bias, const
     auto pair_config = [&](cudaLaunchConfig_t& cfg, cudaLaunchAttribute* attr, unsigned grid, size_t bytes) {
         cfg = cudaLaunchConfig_t{};
         cfg.gridDim = dim3(grid);
-        cfg.blockDim = dim3(gemm::kThreads);
+        cfg.blockDim = dim3(kThreads);
         cfg.dynamicSmemBytes = bytes;
         cfg.stream = static_cast<cudaStream_t>(stream);
         attr[0].id = cudaLaunchAttributeClusterDimension;
@@ -536,8 +666,7 @@ extern "C" int b2kv_matmul(const void* a, const void* w, const void* bias, const
         cfg.numAttrs = 1;
     };
     if (!configured[dev]) {
-        B2KV_CUDA_TRY(cudaFuncSetAttribute(gemm::gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                           static_cast<int>(smem)));
+        B2KV_CUDA_TRY(cudaFuncSetAttribute(single, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
         B2KV_CUDA_TRY(cudaFuncSetAttribute(pair64, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem_pair)));
         B2KV_CUDA_TRY(cudaFuncSetAttribute(pair128, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem_pair128)));
         B2KV_CUDA_TRY(cudaDeviceGetAttribute(&sm_count[dev], cudaDevAttrMultiProcessorCount, dev));
@@ -558,16 +687,15 @@ extern "C" int b2kv_matmul(const void* a, const void* w, const void* bias, const
     // tiles pay off from a few hundred rows on.
     const int variant = tune_get("gemm_variant");
     const bool pairs_fill = 2 * max_clusters[dev] >= sm_count[dev] - 8;
-    const bool use_pair =
-        max_clusters[dev] > 0 && (variant == 2 || variant == 3 || (variant == 0 && pairs_fill && M > 2 * gemm::kBM));
+    const bool use_pair = max_clusters[dev] > 0 && (variant == 2 || variant == 3 || (variant == 0 && pairs_fill && tall));
     if (use_pair) {
-        p.tiles_m = static_cast<int>((static_cast<long long>(M) + 2 * gemm::kBM - 1) / (2 * gemm::kBM));
-        const long long clusters = std::min<long long>(static_cast<long long>(p.tiles_m) * p.tiles_n, max_clusters[dev]);
+        p.tiles_m = static_cast<int>(max_tiles_m_pair);
+        const long long clusters = std::min<long long>(max_tiles_m_pair * tiles_n, max_clusters[dev]);
         cudaLaunchConfig_t cfg;
         cudaLaunchAttribute attr[1];
         if (variant != 2) {  // default: 128 input features per stage (half as many barrier round trips per flop)
             CUtensorMap tw128;
-            if (!gemm::make_map(&tw128, w, K, N, 128)) return B2KV_ERR_UNSUPPORTED;
+            if (!make_map(&tw128, w, w_rows, p.N, ldw, 128)) return B2KV_ERR_UNSUPPORTED;
             pair_config(cfg, attr, static_cast<unsigned>(2 * clusters), smem_pair128);
             B2KV_CUDA_TRY(cudaLaunchKernelEx(&cfg, pair128, ta, tw128, p));
         } else {
@@ -577,8 +705,54 @@ extern "C" int b2kv_matmul(const void* a, const void* w, const void* bias, const
         B2KV_CUDA_TRY(cudaGetLastError());
         return B2KV_OK;
     }
-    const long long grid = std::min<long long>(tiles_m * tiles_n, sm_count[dev]);
-    gemm::gemm_tc_kernel<<<static_cast<unsigned>(grid), gemm::kThreads, smem, static_cast<cudaStream_t>(stream)>>>(ta, tw, p);
+    const long long grid = std::min<long long>(max_tiles_m * tiles_n, sm_count[dev]);
+    single<<<static_cast<unsigned>(grid), kThreads, smem, static_cast<cudaStream_t>(stream)>>>(ta, tw, p);
     B2KV_CUDA_TRY(cudaGetLastError());
     return B2KV_OK;
+}
+
+}  // namespace gemm
+
+}  // namespace b2kv
+
+using namespace b2kv;
+
+extern "C" int b2kv_matmul(const void* a, const void* w, const void* bias, const void* residual, void* out, int M, int K,
+                           int N, int activation, int dtype, int32_t* dev_status, void* stream) {
+    if (dtype != B2KV_DTYPE_BF16) return B2KV_ERR_UNSUPPORTED;
+    if (!a || !w || !out) return B2KV_ERR_BAD_ARG;
+    if (M <= 0 || K <= 0 || N <= 0 || activation < 0 || activation > 1) return B2KV_ERR_BAD_ARG;
+    // row pitches must be multiples of 16 bytes (tensor maps, 16-byte epilogue accesses)
+    if (K % 8 != 0 || N % 8 != 0) return B2KV_ERR_UNSUPPORTED;
+    if (!aligned16(a) || !aligned16(w) || !aligned16(out) || !aligned16(residual) || !aligned16(bias)) return B2KV_ERR_ALIGN;
+    const long long tiles_m = (static_cast<long long>(M) + gemm::kBM - 1) / gemm::kBM;
+    gemm::GemmParams p{static_cast<const __nv_bfloat16*>(bias), static_cast<const __nv_bfloat16*>(residual),
+                       static_cast<__nv_bfloat16*>(out), M, N, K, activation, 0, 0, dev_status};
+    return gemm::launch(p, a, M, K, w, K, N, tiles_m, (tiles_m + 1) / 2, M > 2 * gemm::kBM, stream);
+}
+
+// b2kv_linear with many rows: one product, or rows grouped by expert.
+int b2kv::linear_tiled_tc(const b2kv_linear_args& a, int32_t* dev_status, void* stream) {
+    if (a.dtype != B2KV_DTYPE_BF16) return B2KV_ERR_UNSUPPORTED;
+    const bool grouped = a.group_rows != nullptr;
+    if (a.groups > 1 && !grouped) return B2KV_ERR_UNSUPPORTED;
+    if (grouped && (a.groups > gemm::kMaxGroups || a.group_w != static_cast<int64_t>(a.K) * a.ld_w)) return B2KV_ERR_UNSUPPORTED;
+    if (!aligned16(a.x) || !aligned16(a.w) || a.ld_x % 8 || a.ld_w % 8 || a.ld_x < a.K || a.ld_w < a.N) return B2KV_ERR_UNSUPPORTED;
+    int first = 0;
+    for (int s = 0; s < a.n_seg; ++s) {  // 16-byte accesses in the epilogue; 32 columns lie in one segment
+        const b2kv_segment& sg = a.seg[s];
+        const bool f32 = sg.kind == B2KV_SEG_F32, glu = sg.kind >= B2KV_SEG_GLU_SILU;
+        if (first % 32 != 0 || (sg.end - first) % (glu ? 16 : (f32 ? 4 : 8)) != 0) return B2KV_ERR_UNSUPPORTED;
+        if (!aligned16(sg.out) || sg.ld % (f32 ? 4 : 8) != 0) return B2KV_ERR_UNSUPPORTED;
+        first = sg.end;
+    }
+    if (a.residual && (!aligned16(a.residual) || a.ld_residual % 4 != 0)) return B2KV_ERR_UNSUPPORTED;
+    gemm::SegParams p{a, a.rows, a.N, a.K, 0, 0, dev_status};
+    // with groups the number of tiles is only known on the device: every group may end in a partly filled tile
+    const long long part = grouped ? a.groups : 0;
+    const long long tiles_m = (static_cast<long long>(a.rows) + gemm::kBM - 1) / gemm::kBM + part;
+    const long long tiles_m_pair = (static_cast<long long>(a.rows) + 2 * gemm::kBM - 1) / (2 * gemm::kBM) + part;
+    const bool tall = grouped ? a.rows / a.groups > 2 * gemm::kBM : a.rows > 2 * gemm::kBM;
+    return gemm::launch(p, a.x, a.rows, a.ld_x, a.w, grouped ? static_cast<int64_t>(a.groups) * a.K : a.K, a.ld_w, tiles_m,
+                        tiles_m_pair, tall, stream);
 }

@@ -105,6 +105,23 @@ static int launch_simt(const b2kv_linear_args& a, void* stream) {
     return B2KV_OK;
 }
 
+// A per-head product of many rows: the weight-streaming kernel on 128 rows at a time (the heads' matrices are small and
+// stay in L2).
+static int rows_in_slices(const b2kv_linear_args& all, int32_t* dev_status, void* stream) {
+    const int es = elt_bytes(all.dtype);
+    for (int r0 = 0; r0 < all.rows; r0 += 128) {
+        b2kv_linear_args a = all;
+        a.rows = all.rows - r0 < 128 ? all.rows - r0 : 128;
+        a.x = static_cast<const char*>(all.x) + r0 * all.ld_x * es;
+        if (all.residual) a.residual = all.residual + r0 * all.ld_residual;
+        for (int s = 0; s < a.n_seg; ++s)
+            a.seg[s].out = static_cast<char*>(all.seg[s].out) + r0 * all.seg[s].ld * (all.seg[s].kind == B2KV_SEG_F32 ? 4 : es);
+        const int rc = linear_rows_tc(a, dev_status, stream);
+        if (rc != B2KV_OK) return rc;
+    }
+    return B2KV_OK;
+}
+
 }  // namespace lin
 }  // namespace b2kv
 
@@ -128,8 +145,14 @@ extern "C" int b2kv_linear(const b2kv_linear_args* args, int32_t* dev_status, vo
     if (a.path == 2) return linear_rows_tc(a, dev_status, stream);
     if (a.path == 3) return linear_tiled_tc(a, dev_status, stream);
     if (a.path == 0 && a.dtype == B2KV_DTYPE_BF16) {
-        const int rc = (a.group_rows ? a.max_group_rows : a.rows) <= 128 ? linear_rows_tc(a, dev_status, stream)
-                                                                         : linear_tiled_tc(a, dev_status, stream);
+        int rc;
+        if ((a.group_rows ? a.max_group_rows : a.rows) <= 128) {
+            rc = linear_rows_tc(a, dev_status, stream);
+        } else if (a.groups > 1 && a.group_rows == nullptr) {
+            rc = lin::rows_in_slices(a, dev_status, stream);
+        } else {
+            rc = linear_tiled_tc(a, dev_status, stream);
+        }
         if (rc != B2KV_ERR_UNSUPPORTED) return rc;
     }
     return lin::launch_simt(a, stream);
