@@ -449,6 +449,24 @@ int b2kv_latent_decode(const void* q_latent, const void* q, int64_t ld_q, int di
                        int path, void* workspace, size_t workspace_bytes, int32_t* dev_status, void* stream);
 
 /*
+ * Attention of prompt portions over keys and values expanded from the cached latent rows (bf16, tensor cores).  Query row i
+ * of a segment (rows row0 .. row0 + n - 1 of the step) sits at key row own + i of that segment and sees the `window` key rows
+ * up to its own (window <= 0: all of them).  Key row t of a segment is row kv_row0 + t of `keys` and `values` (heads side by side,
+ * pitch ld_kv; dim and vdim elements per head) and row cache_row0 + t of key_cache [cache_rows, rot] (the rotated part all heads
+ * share).  q as b2kv_latent_append leaves it; out [rows, >= H * vdim].  A row block is 256 query rows of one segment:
+ * first_block counts the blocks of the segments before, n_blocks those of all.  `segments` is a device array.
+ * b2kv_latent_prefill_supported says whether the sizes have this form (dim <= 128, rot <= 64, vdim <= 128, multiples of 8).
+ */
+typedef struct b2kv_prompt_segment {
+    int32_t row0, n, kv_row0, cache_row0, own, first_block;
+} b2kv_prompt_segment;
+int b2kv_latent_prefill_supported(int dim, int rot, int vdim, int kv_rank, int dtype);
+int b2kv_latent_prefill(const void* q, int64_t ld_q, const void* keys, const void* values, int64_t ld_kv, const void* key_cache,
+                        int64_t cache_rows, void* out, int64_t ld_out, const b2kv_prompt_segment* segments, int n_segments,
+                        int n_blocks, int rows, int kv_rows, int H, int dim, int rot, int vdim, int window, float scale, int dtype,
+                        int32_t* dev_status, void* stream);
+
+/*
  * Mixture of experts.  b2kv_route: per row of logits [rows, ld] (fp32, `experts` of them used): softmax over all experts,
  * the `keep` best of `groups` equal groups by their largest score, the `top` best experts of those (lowest index among
  * equals); expert ids and scores go to idx / score [rows, top], and the experts' row counts to counts (int32[2 * experts]:

@@ -102,6 +102,9 @@ SIGNATURES = {
     "b2kv_latent_decode_workspace_bytes": (_sz, [_i, _i, _i, _i, _i]),
     "b2kv_latent_decode": (_i, [_vp, _vp, _i64, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp,
                                 _sz, _vp, _vp]),
+    "b2kv_latent_prefill_supported": (_i, [_i, _i, _i, _i, _i]),
+    "b2kv_latent_prefill": (_i, [_vp, _i64, _vp, _vp, _i64, _vp, _i64, _vp, _i64, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i,
+                                 _vp, _vp]),
     "b2kv_route": (_i, [_vp, _i64, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp]),
     "b2kv_moe_plan": (_i, [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _i64, _vp, _i64, _i, _i, _vp]),
     "b2kv_moe_combine": (_i, [_vp, _i64, _vp, _i64, _vp, _vp, _i, _i, _i, _i, _vp]),

@@ -430,6 +430,7 @@ __device__ __forceinline__ void epilogue_rows(const SegParams& p, uint32_t t_add
         const int col0 = col_base + c * 32;
         if (col0 >= p.N) break;
         uint32_t acc[32];
+        __syncwarp();  // lanes past row_end skipped the stores of the columns before
         tmem_ld32(t_addr + c * 32, acc);
         const int s = lin::segment_of(p.a, col0);
         const b2kv_segment& sg = p.a.seg[s];

@@ -299,6 +299,7 @@ linear_rows_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
             const uint32_t t_lane = sm.tmem_base + (static_cast<uint32_t>(warp * 32) << 16);
             for (int nb = 0; nb < Bn; nb += 16) {
                 uint32_t v[16];
+                __syncwarp();  // the lanes' stores above differ
                 tmem_ld16(t_lane + nb, v);
                 tmem_wait_ld();
                 float f[16];

@@ -30,7 +30,7 @@ from ._native import lib as _lib
 from ._native import check as _check
 from .batch import batch_begin, batch_commit, batch_op_begin
 from .kv_cache import kv_cache_create
-from .latent import LatentShape, RowPlaces
+from .latent import LatentShape, PromptPlan, RowPlaces
 from .moe import ExpertWeights, MoeScratch, RouterShape
 from .projection import SEG_F32, SEG_GLU_CLAMP, SEG_STORE, OutputSegment, linear
 from .registry import register_model
@@ -221,6 +221,7 @@ class GigezenState:
     seq_lens: torch.Tensor           # int32 [batch_size] on the device, shared by all caches
     lengths: List[int]               # the same on the host
     scratch: Dict[str, torch.Tensor] = field(default_factory=dict)
+    prompt_form: bool = False        # every layer's sizes have a tensor-core form for prompt portions
     logits: Optional[GPUBuffer2D] = None  # fp32 rows of the last step
     layer_tap: Optional[list] = None      # debugging: receives a copy of the residual rows after every layer
 
@@ -261,7 +262,8 @@ def state_create(ctx: GPUContext, cfg: GigezenConfig, weights: GigezenWeights, b
                                                           head_dim=a.rot, v_head_dim=a.kv_rank, dtype=dtype, ragged=True))
             owned[i].seq_lens = seq_lens
     return GigezenState(cfg=cfg, weights=weights, batch_size=batch_size, max_seq_len=max_seq_len, dtype=dtype, owned=owned,
-                        seq_lens=seq_lens, lengths=[0] * batch_size)
+                        seq_lens=seq_lens, lengths=[0] * batch_size,
+                        prompt_form=all(latent.prefill_supported(lc.attention, dtype) for lc in cfg.layers))
 
 
 def state_set_lengths(state: GigezenState, lens: Sequence[int]) -> None:
@@ -287,16 +289,6 @@ def state_release(state: GigezenState, slot: int) -> None:
 # the step
 # ---------------------------------------------------------------------------------------------------------------
 
-@dataclass
-class PromptSpan:
-    """Rows ``row0 .. row0 + n - 1`` of a step: positions ``start ..`` of one sequence, attended as a prompt portion."""
-
-    row0: int
-    n: int
-    slot: int
-    start: int
-
-
 def _sub(b: GPUBuffer2D, r0: int, n: int, c0: int = 0, cols: Optional[int] = None) -> GPUBuffer2D:
     cols = b.shape[1] - c0 if cols is None else cols
     return GPUBuffer2D(buffer=b.buffer[r0:r0 + n, c0:c0 + cols], shape=(n, cols), size=n * cols)
@@ -315,7 +307,7 @@ def _attend_rows(ctx, state: GigezenState, i: int, y: GPUBuffer2D, z: GPUBuffer2
 
 
 def _layer(ctx, state: GigezenState, i: int, x: GPUBuffer2D, places: RowPlaces, n_single: int, span: int,
-           prompts: Sequence[PromptSpan]) -> None:
+           plans: Dict[int, PromptPlan]) -> None:
     lc, w, T = state.cfg.layers[i], state.weights.layers[i], x.shape[0]
     a, cfg, dt = lc.attention, state.cfg, state.dtype
     cache = state.cache_of(i)
@@ -335,8 +327,8 @@ def _layer(ctx, state: GigezenState, i: int, x: GPUBuffer2D, places: RowPlaces, 
     if n_single:
         head_places = RowPlaces(None if places.slot is None else places.slot[:n_single], places.pos[:n_single])
         _attend_rows(ctx, state, i, _sub(y, 0, n_single), _sub(z, 0, n_single, 0, a.heads * a.vdim), head_places, span)
-    for p in prompts:
-        _attend_prompt(ctx, state, i, _sub(y, p.row0, p.n), _sub(z, p.row0, p.n, 0, a.heads * a.vdim), p)
+    if plans:
+        _attend_prompts(ctx, state, i, y, _sub(z, 0, T, 0, a.heads * a.vdim), plans[a.window])
     linear(ctx, z, w.w_out, w.a_cols + w.ff_cols, [OutputSegment(cfg.width, SEG_F32, x)], residual=x)
     if lc.router:
         moe.moe_feed_forward(ctx, h, logits, w.experts, lc.router, _moe_scratch(state, lc, w, T), x)
@@ -354,18 +346,27 @@ def _moe_scratch(state: GigezenState, lc: LayerConfig, w: LayerWeights, T: int) 
                       m=state.rows(f"moe_m{w.experts.ff}", n, w.experts.ff, dt), y=state.rows("moe_y", n, width, dt))
 
 
-def _attend_prompt(ctx, state: GigezenState, i: int, y: GPUBuffer2D, z: GPUBuffer2D, p: PromptSpan) -> None:
-    raise NotImplementedError
+def _attend_prompts(ctx, state: GigezenState, i: int, y: GPUBuffer2D, z: GPUBuffer2D, plan: PromptPlan) -> None:
+    """Attention of prompt portions: their visible latents become keys and values of all heads in one product."""
+    a, w, cache = state.cfg.layers[i].attention, state.weights.layers[i], state.cache_of(i)
+    cols = w.k_cols + a.heads * a.vdim
+    kv = state.rows(f"kv{cols}", plan.kv_rows, cols, state.dtype)
+    latents = cache.layers[0].v_cache.buffer.view(-1, a.kv_rank)
+    for _, _, cache_row, visible, kv_row in plan.portions:
+        linear(ctx, _b2(latents[cache_row:cache_row + visible]), w.expand, a.kv_rank,
+               [OutputSegment(cols, SEG_STORE, _sub(kv, kv_row, visible))])
+    latent.latent_prefill(ctx, y, _sub(kv, 0, plan.kv_rows, 0, a.heads * a.dim), _sub(kv, 0, plan.kv_rows, w.k_cols), a, plan,
+                          cache, z)
 
 
 def _run(ctx, state: GigezenState, ids: torch.Tensor, places: RowPlaces, rows: int, n_single: int, span: int,
-         prompts: Sequence[PromptSpan], row_index: Optional[torch.Tensor], n_out: int) -> None:
+         plans: Dict[int, PromptPlan], row_index: Optional[torch.Tensor], n_out: int) -> None:
     """Embedding, all layers and, for the ``n_out`` rows of ``row_index`` (None: all), the logits."""
     cfg, w = state.cfg, state.weights
     x = state.rows("x", rows, cfg.width, torch.float32)
     embedding_rows(ctx, w.embedding, ids, x)
     for i in range(len(cfg.layers)):
-        _layer(ctx, state, i, x, places, n_single, span, prompts)
+        _layer(ctx, state, i, x, places, n_single, span, plans)
     if n_out == 0:
         return
     hl = state.rows("h_out", n_out, cfg.width, state.dtype)
@@ -383,7 +384,7 @@ def decode_step(ctx: GPUContext, state: GigezenState, token_ids: GPUBuffer1D, ne
     if upper >= state.max_seq_len:
         raise ValueError(f"Cache is full: current_len={upper}, max_seq_len={state.max_seq_len}")
     B = state.batch_size
-    _run(ctx, state, token_ids.buffer, RowPlaces(None, state.seq_lens), B, B, upper + 1, (), None, B)
+    _run(ctx, state, token_ids.buffer, RowPlaces(None, state.seq_lens), B, B, upper + 1, {}, None, B)
     if next_ids is not None:
         argmax(ctx, state.logits, next_ids)
     _check(_lib.b2kv_advance_lengths(state.seq_lens.data_ptr(), B, 1, batch_op_begin(ctx)))
@@ -405,9 +406,9 @@ def forward(ctx: GPUContext, state: GigezenState, entries: Sequence[Tuple[int, S
             raise ValueError("an entry needs at least one token")
         if state.lengths[slot] + len(tokens) > state.max_seq_len:
             raise ValueError(f"Cache is full: current_len={state.lengths[slot]} + {len(tokens)}, max_seq_len={state.max_seq_len}")
-    short = [len(t) <= SHORT_ENTRY or not _prompt_form(state) for _, t, _ in entries]
+    short = [len(t) <= SHORT_ENTRY or not state.prompt_form for _, t, _ in entries]
     order = sorted(range(len(entries)), key=lambda j: not short[j])  # stable: short entries first
-    ids, slots, pos, first_row, prompts, lens = [], [], [], {}, [], list(state.lengths)
+    ids, slots, pos, first_row, spans, lens = [], [], [], {}, [], list(state.lengths)
     n_single, span = 0, 1
     for j in order:
         slot, tokens, _ = entries[j]
@@ -417,29 +418,28 @@ def forward(ctx: GPUContext, state: GigezenState, entries: Sequence[Tuple[int, S
             n_single += n
             span = max(span, start + n)
         else:
-            prompts.append(PromptSpan(row0=len(ids), n=n, slot=slot, start=start))
+            spans.append((len(ids), n, slot, start))
         ids += [int(t) for t in tokens]
         slots += [slot] * n
         pos += range(start, start + n)
         lens[slot] = start + n
     want = [first_row[j] + int(p) for j in range(len(entries)) for p in entries[j][2]]
     T, n_out = len(ids), len(want)
-    # one upload per step: ids, sequences, positions, wanted rows, lengths behind the step
-    host = torch.tensor(ids + slots + pos + want + lens, dtype=torch.int32).pin_memory()
-    meta = host.to(ctx.device, non_blocking=True)
-    places = RowPlaces(meta[T:2 * T], meta[2 * T:3 * T])
+    windows = sorted({lc.attention.window for lc in state.cfg.layers}) if spans else []
+    plans = {win: PromptPlan.build(spans, win, state.max_seq_len) for win in windows}
+    # one upload per step: ids, sequences, positions, wanted rows, lengths behind the step, prompt tables
+    parts = [ids, slots, pos, want, lens] + [plans[win].rows() for win in windows]
+    host = torch.tensor([v for part in parts for v in part], dtype=torch.int32).pin_memory()
+    pieces = list(host.to(ctx.device, non_blocking=True).split([len(part) for part in parts]))
+    for win, table in zip(windows, pieces[5:]):
+        plans[win].table = table
     batch_begin(ctx)
-    _run(ctx, state, meta[:T], places, T, n_single, span, prompts, meta[3 * T:3 * T + n_out], n_out)
+    _run(ctx, state, pieces[0], RowPlaces(pieces[1], pieces[2]), T, n_single, span, plans, pieces[3], n_out)
     batch_commit(ctx)
-    state.seq_lens.copy_(meta[3 * T + n_out:])
+    state.seq_lens.copy_(pieces[4])
     state.lengths = lens
     state._sync_upper_bound()
     return state.logits.buffer if n_out else None
-
-
-def _prompt_form(state: GigezenState) -> bool:
-    """Whether the layers' shapes have a tensor-core form for prompt portions."""
-    return False
 
 
 # ---------------------------------------------------------------------------------------------------------------

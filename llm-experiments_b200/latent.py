@@ -89,3 +89,54 @@ def latent_decode(ctx: GPUContext, q_latent: GPUBuffer2D, y: GPUBuffer2D, shape:
         places.slot_ptr(), places.pos.data_ptr(), cache.batch_size, cache.max_seq_len, rows, shape.heads, shape.kv_rank,
         shape.rot, shape.window, span, shape.scale, dt, path, None if ws is None else ws.data_ptr(),
         0 if ws is None else ws.numel(), dev_status_ptr(ctx), stream))
+
+
+@dataclass
+class PromptPlan:
+    """Prompt portions of one step for layers with one window: per portion its rows of the step, the visible part of its
+    sequence's cache and where that part is expanded to, and the device table ``latent_prefill`` reads."""
+
+    portions: list          # (row0, n, first cache row, visible rows, first expanded row)
+    table: Optional[torch.Tensor]  # int32 [portions, 6] on the device
+    n_blocks: int
+    kv_rows: int
+
+    BLOCK = 256  # query rows of one block of the kernel
+
+    @staticmethod
+    def build(spans, window: int, max_seq_len: int) -> "PromptPlan":
+        """``spans``: (row0, n, sequence, start position); the table is filled in by ``rows()`` + an upload."""
+        portions, at, blocks = [], 0, 0
+        for row0, n, slot, start in spans:
+            lo = max(0, start - window + 1) if window > 0 else 0
+            portions.append((row0, n, slot * max_seq_len + lo, start + n - lo, at))
+            at += start + n - lo
+            blocks += (n + PromptPlan.BLOCK - 1) // PromptPlan.BLOCK
+        return PromptPlan(portions=portions, table=None, n_blocks=blocks, kv_rows=at)
+
+    def rows(self) -> list:
+        """The table as a flat list of integers (``b2kv_prompt_segment``)."""
+        out, first = [], 0
+        for row0, n, cache_row, visible, kv_row in self.portions:
+            out += [row0, n, kv_row, cache_row, visible - n, first]
+            first += (n + PromptPlan.BLOCK - 1) // PromptPlan.BLOCK
+        return out
+
+
+def prefill_supported(shape: LatentShape, dtype: torch.dtype) -> bool:
+    return shape.scale > 0 and bool(_native.lib.b2kv_latent_prefill_supported(shape.dim, shape.rot, shape.vdim, shape.kv_rank,
+                                                                             dtype_code(dtype)))
+
+
+@reference_op("latent_prefill")
+def latent_prefill(ctx: GPUContext, y: GPUBuffer2D, keys: GPUBuffer2D, values: GPUBuffer2D, shape: LatentShape,
+                   plan: PromptPlan, cache: KVCache, out: GPUBuffer2D) -> None:
+    """Attention of prompt portions: ``y`` and ``out`` are the step's rows, ``keys`` ``[kv_rows, heads * dim]`` and ``values``
+    ``[kv_rows, heads * vdim]`` (views of one buffer) the expanded visible rows of the plan's portions."""
+    key, _ = _latent_cache(cache, shape)
+    stream = batch_op_begin(ctx)
+    _native.check(_native.lib.b2kv_latent_prefill(
+        y.buffer.data_ptr(), y.buffer.stride(0), keys.buffer.data_ptr(), values.buffer.data_ptr(), keys.buffer.stride(0), key,
+        cache.batch_size * cache.max_seq_len, out.buffer.data_ptr(), out.buffer.stride(0), plan.table.data_ptr(),
+        len(plan.portions), plan.n_blocks, y.shape[0], plan.kv_rows, shape.heads, shape.dim, shape.rot, shape.vdim, shape.window,
+        shape.scale, dtype_code(y.buffer.dtype), dev_status_ptr(ctx), stream))
