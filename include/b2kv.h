@@ -437,10 +437,10 @@ int b2kv_latent_append(void* y, int64_t ld_y, int H, int dim, int rot, int rot_d
  *   score_t = (q_latent[i, h, :] . latent[t, :] + q[i, h, dim:] . key[t, :]) * scale,  t in (row_pos[i] - window, row_pos[i]]
  *   out[i, h, :] = sum_t softmax(score)_t latent[t, :]
  * q_latent [rows, H, kv_rank] is the unrotated query carried into the latent space; window <= 0 sees every earlier token.
- * span is an upper bound of the tokens a row sees.  The rows' own tokens are in the cache already.  bf16 with kv_rank a
- * multiple of 64 up to 512, rot a multiple of 16 up to 64 and H up to 128 runs on the tensor cores (split over the window, partial results
- * merged by the CTA that finishes a row last; workspace of b2kv_latent_decode_workspace_bytes bytes, zeroed once before
- * its first use), everything else on CUDA cores.  path: 0 = choose, 1 = CUDA cores, 2 = tensor cores.
+ * span is an upper bound of the tokens a row sees.  The rows' own tokens are in the cache already.  bf16 with dim,
+ * kv_rank and rot multiples of 8, kv_rank up to 512 and rot up to 64 runs on the tensor cores (few rows are split over their
+ * windows, whose partial results go to a workspace of b2kv_latent_decode_workspace_bytes bytes), everything else on CUDA
+ * cores (kv_rank up to 1024).  path: 0 = choose, 1 = CUDA cores, 2 = tensor cores.
  */
 size_t b2kv_latent_decode_workspace_bytes(int rows, int H, int kv_rank, int span, int dtype);
 int b2kv_latent_decode(const void* q_latent, const void* q, int64_t ld_q, int dim, const void* key_cache,

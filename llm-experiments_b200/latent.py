@@ -81,7 +81,7 @@ def latent_decode(ctx: GPUContext, q_latent: GPUBuffer2D, y: GPUBuffer2D, shape:
     span = min(span, shape.window) if shape.window > 0 else span
     nbytes = _native.lib.b2kv_latent_decode_workspace_bytes(rows, shape.heads, shape.kv_rank, span, dt) if path != 1 else 0
     if nbytes and (cache.workspace is None or cache.workspace.numel() < nbytes):
-        cache.workspace = torch.zeros(nbytes, dtype=torch.uint8, device=ctx.device)
+        cache.workspace = torch.empty(nbytes, dtype=torch.uint8, device=ctx.device)
     ws = cache.workspace if nbytes else None
     stream = batch_op_begin(ctx)
     _native.check(_native.lib.b2kv_latent_decode(
