@@ -10,6 +10,7 @@ import pathlib
 
 _PKG = pathlib.Path(__file__).resolve().parent
 LIB_PATH = _PKG / "libb2kv.so"
+SERVE_LIB_PATH = _PKG / "libb2kv_serve.so"  # the part models are served with (build.py --serve), where that is all there is
 
 DTYPE_F32 = 0
 DTYPE_BF16 = 1
@@ -120,15 +121,26 @@ class B2KVError(RuntimeError):
         self.status = status
 
 
+def _not_built(name: str):
+    def call(*_):
+        raise ImportError(f"{name} is not part of {SERVE_LIB_PATH.name}; build the whole library with {_PKG.name}/build.py")
+
+    return call
+
+
 def _load() -> ctypes.CDLL:
-    if not LIB_PATH.exists():
+    path = LIB_PATH if LIB_PATH.exists() or not SERVE_LIB_PATH.exists() else SERVE_LIB_PATH
+    if not path.exists():
         raise ImportError(
             f"{LIB_PATH} is missing. Build the CUDA library first: "
             f"`python {_PKG.name}/build.py` (needs nvcc with sm_100a support). "
             "This package has no CPU fallback."
         )
-    lib = ctypes.CDLL(str(LIB_PATH))
+    lib = ctypes.CDLL(str(path))
     for name, (restype, argtypes) in SIGNATURES.items():
+        if path == SERVE_LIB_PATH and not hasattr(lib, name):
+            setattr(lib, name, _not_built(name))
+            continue
         fn = getattr(lib, name)  # AttributeError here means header and library disagree
         fn.restype = restype
         fn.argtypes = argtypes

@@ -1,8 +1,12 @@
 """Build ``libb2kv.so`` (the C-ABI CUDA library) in-tree with nvcc for sm_100a.
 
-``python llm-experiments_b200/build.py [--force] [--verbose]``.  The library has no
+``python llm-experiments_b200/build.py [--force] [--verbose] [--serve]``.  The library has no
 dependency on torch or Python: it is loaded with ctypes.  Sources are compiled to
 objects in parallel and linked with the static CUDA runtime.
+
+``--serve`` builds ``libb2kv_serve.so`` instead: only what models with a 32-bit residual stream are served with, a
+fraction of the compile time (the decode-attention and prefill variants of the reference path take most of it).  It is
+loaded where the whole library has not been built.
 """
 from __future__ import annotations
 
@@ -16,7 +20,10 @@ PKG = pathlib.Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 INCLUDE = PKG.parent / "include"
 OUT = PKG / "libb2kv.so"
+SERVE_OUT = PKG / "libb2kv_serve.so"
 OBJ_DIR = PKG / "build"
+SERVE_SOURCES = ("api", "append", "gemm", "latent", "latent_decode_tc", "latent_prefill", "linear", "linear_rows", "moe", "rows",
+                 "step_tail")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -31,8 +38,8 @@ def _nvcc() -> str:
     return cand if os.path.exists(cand) else "nvcc"
 
 
-def sources():
-    return sorted(CSRC.glob("*.cu"))
+def sources(serve: bool = False):
+    return [f for f in sorted(CSRC.glob("*.cu")) if not serve or f.stem in SERVE_SOURCES]
 
 
 def _newest_input() -> float:
@@ -40,13 +47,14 @@ def _newest_input() -> float:
     return max(f.stat().st_mtime for f in files)
 
 
-def up_to_date() -> bool:
-    return OUT.exists() and OUT.stat().st_mtime >= _newest_input()
+def up_to_date(out: pathlib.Path = OUT) -> bool:
+    return out.exists() and out.stat().st_mtime >= _newest_input()
 
 
-def build(force: bool = False, verbose: bool = False) -> pathlib.Path:
-    if not force and up_to_date():
-        return OUT
+def build(force: bool = False, verbose: bool = False, serve: bool = False) -> pathlib.Path:
+    out = SERVE_OUT if serve else OUT
+    if not force and up_to_date(out):
+        return out
     OBJ_DIR.mkdir(exist_ok=True)
     extra = ["-Xptxas", "-v"] if verbose else []
 
@@ -61,11 +69,11 @@ def build(force: bool = False, verbose: bool = False) -> pathlib.Path:
         return obj
 
     with concurrent.futures.ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 1)) as pool:
-        objs = list(pool.map(compile_one, sources()))
-    link = [_nvcc(), "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", str(OUT), *map(str, objs)]
+        objs = list(pool.map(compile_one, sources(serve)))
+    link = [_nvcc(), "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", str(out), *map(str, objs)]
     subprocess.run(link, check=True)
-    return OUT
+    return out
 
 
 if __name__ == "__main__":
-    print(build(force="--force" in sys.argv, verbose="--verbose" in sys.argv))
+    print(build(force="--force" in sys.argv, verbose="--verbose" in sys.argv, serve="--serve" in sys.argv))

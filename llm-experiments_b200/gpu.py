@@ -29,8 +29,11 @@ from .kv_cache import (
     kv_cache_set_lengths,
     kv_cache_update,
 )
-from .projection import matmul, qkv_project_append
-from .step_tail import argmax, embedding, extract_last_tokens, layernorm, softmax
+from .latent import latent_append, latent_decode, latent_prefill
+from .moe import moe_feed_forward
+from .projection import linear, matmul, qkv_project_append
+from .registry import architectures, load_model
+from .step_tail import argmax, embedding, embedding_rows, extract_last_tokens, layernorm, rms_norm, softmax
 from .types import GPUBuffer1D, GPUBuffer2D, GPUConfig, GPUContext, KVCache, KVCacheConfig, KVCacheLayer
 
 __all__ = [
@@ -46,4 +49,7 @@ __all__ = [
     "kv_cache_gather", "kv_cache_set_lengths",
     "embedding", "layernorm", "extract_last_tokens", "softmax", "argmax",
     "qkv_project_append", "matmul",
+    # extensions: building blocks of decoders with a 32-bit residual stream, and models from folders
+    "linear", "embedding_rows", "rms_norm", "latent_append", "latent_decode", "latent_prefill", "moe_feed_forward",
+    "architectures", "load_model",
 ]

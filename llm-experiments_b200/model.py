@@ -27,6 +27,7 @@ from .batch import batch_begin, batch_commit
 from .decode_layer import DecoderLayerScratch, DecoderLayerWeights, PromptLayerScratch
 from .kv_cache import kv_cache_create, kv_cache_reset
 from .projection import matmul
+from .registry import register_model
 from .step_tail import argmax, embedding, extract_last_tokens, layernorm
 from .types import GPUBuffer1D, GPUBuffer2D, GPUContext, KVCache, KVCacheConfig
 
@@ -217,7 +218,10 @@ class GraphedDecodeStep:
     ``token_ids`` (or pass ``feed_back=True`` to copy ``next_ids`` there on the device after every step).
     """
 
-    def __init__(self, ctx: GPUContext, state: DecoderState, feed_back: bool = False):
+    def __init__(self, ctx: GPUContext, state: DecoderState, feed_back: bool = False, step_fn=None):
+        """``step_fn(ctx, state, token_ids, next_ids)`` is the step to capture; ``decode_step`` unless another model's state
+        (anything with ``batch_size`` and ``caches``) brings its own."""
+        self.step_fn = step_fn or decode_step
         if any(c.seq_lens is None for c in state.caches):
             raise ValueError("a graphed decode step needs per-sequence lengths on the device (ragged=True)")
         self.ctx, self.state, self.feed_back = ctx, state, feed_back
@@ -229,7 +233,7 @@ class GraphedDecodeStep:
     def _record(self) -> None:
         ctx, state = self.ctx, self.state
         batch_begin(ctx)
-        decode_step(ctx, state, self.token_ids, self.next_ids)
+        self.step_fn(ctx, state, self.token_ids, self.next_ids)
         batch_commit(ctx)
         if self.feed_back:
             self.token_ids.buffer.copy_(self.next_ids.buffer)
@@ -243,12 +247,15 @@ class GraphedDecodeStep:
         caches = state.caches
         cap = caches[0].max_seq_len
         keep_len = [c.current_len for c in caches]
+        keep_host = list(getattr(state, "lengths", ()))
         if max(keep_len) >= cap:
             raise ValueError(f"Cache is full: current_len={max(keep_len)}, max_seq_len={cap}")
         keep_dev = [c.seq_lens.clone() for c in caches]
         keep_tok = self.token_ids.buffer.clone()
         side = torch.cuda.Stream(device=ctx.device)
         side.wait_stream(torch.cuda.current_stream(ctx.device))
+        for c in caches:
+            c.current_len = cap - 1
         with torch.cuda.stream(side):
             self._record()  # warm-up: nothing allocates or configures a kernel inside the capture
             for c, n, dev in zip(caches, keep_len, keep_dev):
@@ -264,6 +271,8 @@ class GraphedDecodeStep:
         torch.cuda.current_stream(ctx.device).wait_stream(side)
         for c, n in zip(caches, keep_len):
             c.current_len = n
+        if keep_host:
+            state.lengths = keep_host
         self.graph = graph
 
     def step(self) -> None:
@@ -274,8 +283,11 @@ class GraphedDecodeStep:
         if caches[0].current_len >= caches[0].max_seq_len:
             raise ValueError(f"Cache is full: current_len={caches[0].current_len}, max_seq_len={caches[0].max_seq_len}")
         self.graph.replay()
-        for c in caches:
-            c.current_len += 1
+        if hasattr(self.state, "advance_host"):
+            self.state.advance_host()
+        else:
+            for c in caches:
+                c.current_len += 1
 
 
 class CachedDecoder:
@@ -319,3 +331,19 @@ class _CacheGroup:
     def current_len(self, value: int) -> None:
         for cache in self.state.caches:
             cache.current_len = value
+
+
+@register_model("GPTDecoder")
+def _build(ctx: GPUContext, config: dict, weights: dict, dtype: torch.dtype, batch_size: int, max_tokens: int) -> CachedDecoder:
+    """The decoder of a model folder: ``config`` holds the fields of ``DecoderConfig``, the checkpoint ``embedding``,
+    ``out_proj``, ``lnf_gamma``, ``lnf_beta`` and ``layers.<i>.<name>`` for the fields of ``DecoderLayerWeights``."""
+    if dtype != torch.bfloat16:
+        raise ValueError("this decoder runs in bfloat16 only")
+    if batch_size != 1:
+        raise ValueError("CachedDecoder serves one sequence at a time")
+    cfg = DecoderConfig(**{k: config[k] for k in ("vocab_size", "context_size", "embedding_dim", "n_heads", "n_layers")})
+    get = lambda name: weights[name].float().numpy()  # noqa: E731
+    layers = [{k: get(f"layers.{i}.{k}") for k in DecoderLayerWeights.__dataclass_fields__} for i in range(cfg.n_layers)]
+    params = dict(embedding=get("embedding"), pos_encoding=positional_encoding(cfg.context_size, cfg.embedding_dim), layers=layers,
+                  lnf_gamma=get("lnf_gamma"), lnf_beta=get("lnf_beta"), out_proj=get("out_proj"))
+    return CachedDecoder(ctx, cfg, weights_from_numpy(ctx, cfg, params))
