@@ -94,6 +94,21 @@ WORKLOADS = {
     "model_step_small": dict(kind="model_step", B=8, H=32, D=128, lo=128, hi=1024, layers=4, vocab=32768,
                              desc="the same 4-layer decoder at B=8 with short contexts, len~U[128,1024] seed 0: a step is "
                                   "bound by its 36 launches, so it is also timed as one replayed CUDA graph"),
+    "gigezen_decode": dict(kind="gigezen", phase="decode", B=64, lo=512, hi=8192, width=4096, heads=32, ff=10880, layers=4,
+                           experts=64, top=6, expert_ff=1408, window=4096, vocab=32768,
+                           desc="one cached decode step of a 4-layer Gigezen model (width 4096, 32 heads of 128 + 64, latent 512, window "
+                                "4096; dense layers of 3 x 4096 x 10880 and mixtures of 64 experts of 1408, top 6; every second layer "
+                                "reads the latents of the one before): B=64, len~U[512,8192] seed 0"),
+    "gigezen_decode_small": dict(kind="gigezen", phase="decode", B=8, lo=128, hi=1024, width=2048, heads=16, ff=5440, layers=4,
+                                 experts=64, top=6, expert_ff=1408, window=1024, vocab=32768,
+                                 desc="one cached decode step of a 4-layer Gigezen model of width 2048 (16 heads): B=8, len~U[128,1024]"),
+    "gigezen_prefill": dict(kind="gigezen", phase="prefill", B=8, N=4096, width=4096, heads=32, ff=10880, layers=2, experts=64,
+                            top=6, expert_ff=1408, window=4096, vocab=32768,
+                            desc="prompts of B=8 x N=4096 tokens through 2 layers (one dense, one mixture) of the width-4096 Gigezen "
+                                 "model, window 4096"),
+    "gigezen_prefill_small": dict(kind="gigezen", phase="prefill", B=2, N=2048, width=2048, heads=16, ff=5440, layers=2, experts=64,
+                                  top=6, expert_ff=1408, window=1024, vocab=32768,
+                                  desc="prompts of B=2 x N=2048 tokens through 2 layers of a width-2048 Gigezen model, window 1024"),
 }
 SLACK = 1024  # rows of head-room above the longest sequence for the appended tokens
 
@@ -1039,7 +1054,230 @@ def run_model_step(h: Harness, w):
     }
 
 
-RUNNERS = {"prefill": run_prefill, "qkv": run_qkv_append, "layer_step": run_decode_layer,
+def gigezen_config(w):
+    """config.json of the benchmark's model: dense layers with latents of their own, mixtures that read them."""
+    dim, rot, vdim, rank = 128, 64, 128, 512
+    layers = []
+    for i in range(w["layers"]):
+        mixer = dict(heads=w["heads"], dim=dim, rot_dim=rot, vdim=vdim, kv_rank=rank, scale=(dim + rot) ** -0.5,
+                     rot=dict(base=10000.0, dims=rot), mask=dict(size=w["window"]))
+        mlp = dict(kind="dense", ff=w["ff"], limit=7.0)
+        if i % 2:
+            mixer["kv_from"] = i - 1
+            mlp = dict(kind="moe", expert=dict(ff=w["expert_ff"]),
+                       router=dict(experts=w["experts"], top=w["top"], groups=dict(count=8, keep=4)))
+        layers.append(dict(type="latent_attention", mixer=mixer, mlp=mlp))
+    return dict(architecture="Gigezen", layers=layers, vocab=w["vocab"], width=w["width"], norm=dict(eps=1e-6))
+
+
+def run_gigezen(h: Harness, w):
+    """A Gigezen model with random weights: a whole decode step (generated tokens/s, HBM roofline over every weight once and the
+    latents attended) or whole prompts (prompt tokens/s, tensor roofline), and every kernel of the design timed alone on the
+    model's own buffers, each with its roofline.  Kernels whose operands fit L2 are timed over alternating layers only as
+    far as the model has them, and say so."""
+    torch, gpu, ctx = h.torch, h.gpu, h.ctx
+    from llm_experiments_b200 import gigezen, latent, moe
+    from llm_experiments_b200.model import GraphedDecodeStep
+    from llm_experiments_b200.projection import SEG_F32, SEG_GLU_CLAMP, SEG_GLU_SILU, SEG_STORE, OutputSegment, linear
+
+    world, device, decode = h.world, h.device, w["phase"] == "decode"
+    cfg_json = gigezen_config(w)
+    cfg = gigezen.GigezenConfig.from_json(cfg_json)
+    weights = gigezen.prepare_weights(ctx, cfg, gigezen.random_tensors(ctx, cfg_json, seed=7000 + h.rank), torch.bfloat16)
+    h.release()
+    B, width, H, V = w["B"], w["width"], w["heads"], w["vocab"]
+    T_max = (w["hi"] if decode else w["N"]) + 8
+    state = gigezen.state_create(ctx, cfg, weights, B, T_max)
+    gen = torch.Generator(device=device).manual_seed(7100 + h.rank)
+    for c in state.caches:
+        c.layers[0].k_cache.buffer.normal_(generator=gen)
+        c.layers[0].v_cache.buffer.normal_(generator=gen)
+    peak, sustained, burst, kind = measured_peaks()
+    a, dense_w, mix_w = cfg.layers[0].attention, weights.layers[0], weights.layers[1]
+    router = cfg.layers[1].router
+    per_head = H * (a.dim + a.vdim) * a.kv_rank  # key and value matrices
+    dense_params = width * (H * (a.dim + a.rot) + a.kv_rank + a.rot) + per_head + width * H * a.vdim + 3 * width * w["ff"]
+    attn_params = width * H * (a.dim + a.rot) + per_head + width * H * a.vdim
+    expert_params = 3 * width * w["expert_ff"]
+    n_dense, n_mix = (w["layers"] + 1) // 2, w["layers"] // 2
+
+    if decode:
+        lens = make_lengths(w)
+        gigezen.state_set_lengths(state, lens)
+        lens_dev, lens_list = state.seq_lens.clone(), [int(v) for v in lens]
+        tok_b = h.wrap1(torch.randint(0, V, (B,), generator=gen, device=device, dtype=torch.int32))
+        next_b = h.wrap1(torch.empty(B, dtype=torch.int32, device=device))
+        tok_h, next_h = tok_b.buffer.cpu().pin_memory(), torch.empty(B, dtype=torch.int32).pin_memory()
+
+        def rewind():
+            state.seq_lens.copy_(lens_dev)
+            state.lengths = list(lens_list)
+            for c in state.caches:
+                c.current_len = max(lens_list)
+
+        def step_device():
+            rewind()
+            gpu.batch_begin(ctx)
+            gigezen.decode_step(ctx, state, tok_b, next_b)
+            gpu.batch_commit(ctx)
+
+        def step_e2e():
+            gpu.gpu_buffer_1d_write(ctx, tok_h, tok_b)
+            step_device()
+            gpu.gpu_buffer_1d_read(ctx, next_b, next_h)
+
+        rows, tokens, h2d, d2h = B, B, B * 4, B * 4
+    else:
+        N = w["N"]
+        prompts = [np.random.default_rng(s).integers(0, V, size=N).astype(np.int32) for s in range(B)]
+        out_h = torch.empty((B, V), dtype=torch.float32).pin_memory()
+        entries = [(b, prompts[b], [N - 1]) for b in range(B)]
+
+        def step_device():
+            gigezen.state_reset(state)
+            gigezen.forward(ctx, state, entries)
+
+        def step_e2e():
+            step_device()
+            out_h.copy_(state.logits.buffer, non_blocking=True)
+            torch.cuda.current_stream().synchronize()
+
+        rows, tokens, h2d, d2h = B * N, B * N, 3 * B * N * 4, B * V * 4
+
+    sampler = h.sampler()
+    steps = h.steps if decode else min(h.steps, 10)
+    m_step = h.measure(step_device, steps=steps)
+    m_e2e = h.measure(step_e2e, steps=max(2, min(steps, 20)), warmup=1, repeats=min(h.repeats, 3))
+    graph = None
+    if decode:
+        graphed = GraphedDecodeStep(ctx, state, step_fn=gigezen.decode_step)
+        rewind()
+        graphed.capture()
+
+        def step_graph():
+            rewind()
+            graphed.step()
+
+        m_graph = h.measure(step_graph)
+        graph = {"value": world * B / (m_graph["ms"] * 1e-3), "unit": "tokens/s", **spread(m_graph)}
+        rewind()
+
+    # ---- every kernel alone, on the rows, weights and cache of the step above
+    ctx.config.max_batch_operations = 10 ** 9
+    g = torch.Generator(device=device).manual_seed(5)
+    bf = lambda r, c: h.wrap(torch.randn((r, c), generator=g, device=device).to(torch.bfloat16))  # noqa: E731
+    f32 = lambda r, c: h.wrap(torch.randn((r, c), generator=g, device=device))  # noqa: E731
+    view = lambda b, c0, n: h.wrap(b.buffer[:, c0:c0 + n])  # noqa: E731
+    x, hb = f32(rows, width), bf(rows, width)
+    y, z = bf(rows, dense_w.y_cols), bf(rows, dense_w.a_cols + dense_w.ff_cols)
+    cache = state.caches[0]
+    kernels = []
+
+    def kernel(name, fn, flops=0, nbytes=0, note=None):
+        def once():
+            gpu.batch_begin(ctx)
+            fn()
+            gpu.batch_commit(ctx)
+
+        m = h.measure(once, steps=50 if decode else 10, repeats=3)
+        t = m["ms"] * 1e-3
+        need_t, need_b = flops / (sustained * 1e12), nbytes / (peak * 1e9)
+        kernels.append({"kernel": name, "us": 1e3 * m["ms"], "bound": "tensor" if need_t > need_b else "hbm",
+                        "frac": max(need_t, need_b) / t, "TFLOP/s": flops / t / 1e12, "GB/s": nbytes / t / 1e9, **({"note": note} if note else {})})
+
+    n_in, n_out = dense_w.y_cols + 2 * dense_w.ff_cols, dense_w.a_cols + dense_w.ff_cols
+    kernel("rms_norm", lambda: gpu.rms_norm(ctx, x, dense_w.norm, hb, cfg.eps, weight_offset=1.0), 0, rows * width * 6)
+    kernel("linear in (queries, latent, gated hidden rows)", lambda: linear(
+        ctx, hb, dense_w.w_in, width, [OutputSegment(dense_w.y_cols, SEG_STORE, y),
+                                       OutputSegment(n_in, SEG_GLU_CLAMP, view(z, dense_w.a_cols, dense_w.ff_cols))], limit=7.0),
+        2.0 * rows * width * n_in, 2 * (width * n_in + rows * (width + dense_w.y_cols + dense_w.ff_cols)))
+    kernel("linear out (attention and hidden rows onto the residual)", lambda: linear(
+        ctx, z, dense_w.w_out, n_out, [OutputSegment(width, SEG_F32, x)], residual=x), 2.0 * rows * width * n_out,
+        2 * (width * n_out + rows * n_out) + 8 * rows * width)
+    if decode:
+        places = latent.RowPlaces(None, state.seq_lens)
+        ql, ol = bf(rows, H * a.kv_rank), bf(rows, H * a.kv_rank)
+        seen = int(np.minimum(lens + 1, w["window"]).sum())
+        kernel("latent_append", lambda: latent.latent_append(ctx, y, a, dense_w.inv_freq, places, cache, dense_w.latent_norm, cfg.eps), 0,
+               rows * 2 * (2 * dense_w.y_cols + a.kv_rank + a.rot), "latency: a few hundred KB")
+        kernel("linear per head (queries into the latent space)", lambda: linear(
+            ctx, y, dense_w.key_absorb, a.dim, [OutputSegment(a.kv_rank, SEG_STORE, ql, group=a.kv_rank)], groups=H,
+            group_x=a.dim + a.rot, group_w=a.dim * a.kv_rank), 2.0 * rows * H * a.dim * a.kv_rank,
+            2 * (H * a.dim * a.kv_rank + rows * H * (a.dim + a.kv_rank)), "operands stay in L2 (one layer); latency-bound")
+        kernel("latent_decode", lambda: latent.latent_decode(ctx, ql, y, a, places, cache, ol, int(lens.max()) + 1),
+               2.0 * seen * H * (2 * a.kv_rank + a.rot), 2 * (seen * (a.kv_rank + a.rot) + 2 * rows * H * a.kv_rank))
+        kernel("linear per head (values out of the latent space)", lambda: linear(
+            ctx, ol, view(dense_w.expand, dense_w.k_cols, H * a.vdim), a.kv_rank,
+            [OutputSegment(a.vdim, SEG_STORE, view(z, 0, H * a.vdim), group=a.vdim)], groups=H, group_x=a.kv_rank, group_w=a.vdim),
+            2.0 * rows * H * a.vdim * a.kv_rank, 2 * (H * a.vdim * a.kv_rank + rows * H * (a.vdim + a.kv_rank)),
+            "operands stay in L2 (one layer); latency-bound")
+    else:
+        places = latent.RowPlaces(torch.arange(B, device=device, dtype=torch.int32).repeat_interleave(w["N"]).contiguous(),
+                                  torch.arange(w["N"], device=device, dtype=torch.int32).repeat(B))
+        plan = latent.PromptPlan.build([(b * w["N"], w["N"], b, 0) for b in range(B)], w["window"], T_max)
+        plan.table = torch.tensor(plan.rows(), dtype=torch.int32, device=device)
+        cols = dense_w.k_cols + H * a.vdim
+        kv = bf(plan.kv_rows, cols)
+        lat_rows = cache.layers[0].v_cache.buffer.view(-1, a.kv_rank)
+        kernel("latent_append", lambda: latent.latent_append(ctx, y, a, dense_w.inv_freq, places, cache, dense_w.latent_norm, cfg.eps), 0,
+               rows * 2 * (2 * H * a.rot + 2 * (a.kv_rank + a.rot)))
+        kernel("linear (keys and values of one sequence)", lambda: linear(
+            ctx, h.wrap(lat_rows[:w["N"]]), dense_w.expand, a.kv_rank, [OutputSegment(cols, SEG_STORE, h.wrap(kv.buffer[:w["N"]]))]),
+            2.0 * w["N"] * a.kv_rank * cols, 2 * (a.kv_rank * cols + w["N"] * (cols + a.kv_rank)))
+        n = np.arange(w["N"]) + 1
+        pairs = float(np.minimum(n, w["window"]).sum()) * B * H
+        kernel("latent_prefill", lambda: latent.latent_prefill(ctx, y, view(kv, 0, H * a.dim), view(kv, dense_w.k_cols, H * a.vdim), a, plan,
+                                                              cache, view(z, 0, H * a.vdim)), 2.0 * pairs * (a.dim + a.rot + a.vdim),
+               2 * rows * H * (2 * (a.dim + a.vdim) + a.rot))
+    scratch = gigezen._moe_scratch(state, cfg.layers[1], mix_w, rows)
+    logits = f32(rows, mix_w.router_cols)
+    n_sel, e_ff = rows * w["top"], mix_w.experts.ff
+    sub = lambda b: h.wrap(b.buffer[:n_sel])  # noqa: E731
+
+    def route_and_plan():
+        moe.route(ctx, logits, rows, router, scratch)
+        moe.plan(ctx, hb, router, scratch)
+
+    kernel("moe route + plan (3 launches)", route_and_plan, 0, 2 * (rows + n_sel) * width + rows * 4 * router.experts)
+    used = w["experts"] if n_sel > 4 * w["experts"] else int((scratch.offsets.diff() > 0).sum())
+    grouped = dict(groups=w["experts"], group_rows=scratch.offsets, max_group_rows=rows)
+    kernel("linear grouped by expert (gate, up)", lambda: linear(
+        ctx, sub(scratch.sorted_h), mix_w.experts.gate_up, width, [OutputSegment(2 * e_ff, SEG_GLU_SILU, scratch.m)],
+        group_w=width * 2 * e_ff, **grouped), 4.0 * n_sel * width * e_ff, 2 * (used * width * 2 * e_ff + n_sel * (width + e_ff)))
+    kernel("linear grouped by expert (down)", lambda: linear(
+        ctx, sub(scratch.m), mix_w.experts.down, e_ff, [OutputSegment(width, SEG_STORE, scratch.y)], group_w=e_ff * width, **grouped),
+        2.0 * n_sel * width * e_ff, 2 * (used * width * e_ff + n_sel * (width + e_ff)))
+    kernel("moe combine", lambda: moe.combine(ctx, x, router, scratch), 0, 2 * n_sel * width + 8 * rows * width)
+    clocks = sampler.finish()
+    status = int(ctx.dev_status.item()) if ctx.dev_status is not None else 0
+
+    if decode:
+        kv_bytes = w["layers"] * seen * 2 * (a.kv_rank + a.rot)
+        weight_bytes = 2 * (n_dense * dense_params + n_mix * (attn_params + used * expert_params + width * router.experts) + width * V)
+        bound, achieved, peak_v, unit = "hbm", (kv_bytes + weight_bytes) / (m_step["ms"] * 1e-3) / 1e9, peak, "GB/s"
+        extra = {"algorithmic_bytes_per_launch": kv_bytes + weight_bytes, "kv_bytes": kv_bytes, "weight_bytes": weight_bytes}
+    else:
+        gemm = 2.0 * rows * (n_dense * dense_params + n_mix * (attn_params + router.top * expert_params))
+        flops = gemm + w["layers"] * 2.0 * pairs * (a.dim + a.rot + a.vdim) + 2.0 * B * width * V
+        bound, achieved, peak_v, unit = "tensor", flops / (m_step["ms"] * 1e-3) / 1e12, sustained, "TFLOP/s"
+        extra = {"algorithmic_flops_per_launch": flops}
+    launches = (9 * w["layers"] + 8 * n_mix + 5) if decode else ((6 + B) * w["layers"] + 8 * n_mix + 3)
+    return {
+        "metric": "generated tokens/s (whole cached decode step of the model)" if decode else "prompt tokens/s (whole model)",
+        "value": world * tokens / (m_step["ms"] * 1e-3), "unit": "tokens/s", **spread(m_step), "steps": steps, "scaling": "weak",
+        "dtype": "bf16 operands, fp32 accumulation, residual, norms, scores and router",
+        "config": {"workload": w["desc"], "batch_per_gpu": B, "global_batch": world * B,
+                   "l2": "weights and caches far larger than L2, no flush", "parallelism": f"batch-sharded x{world}, no collective"},
+        "e2e": {"value": world * tokens / (m_e2e["ms"] * 1e-3), "unit": "tokens/s", **spread(m_e2e), "h2d_bytes_per_step": h2d,
+                "d2h_bytes_per_step": d2h},
+        "gpu_launches": steps * h.repeats * launches, "gpu_launches_per_step": launches, "clocks": clocks, "dev_status": status,
+        "cuda_graph": graph, "kernels": kernels,
+        "roofline": {"bound": bound, "kernel": "the step's kernels together", "achieved": achieved, "peak": peak_v, "unit": unit,
+                     "frac": achieved / peak_v, "peak_kind": kind, "traffic": None, **extra},
+    }
+
+
+RUNNERS = {"gigezen": run_gigezen, "prefill": run_prefill, "qkv": run_qkv_append, "layer_step": run_decode_layer,
            "prompt_layer": run_prompt_layer, "model_step": run_model_step}
 
 
@@ -1107,7 +1345,7 @@ def run_b200(args):
         "gpu_launches_per_step": head.get("gpu_launches_per_step"), "clocks": head["clocks"],
         "roofline": head["roofline"], "cpu_baseline": head.get("cpu_baseline"),
     }
-    for k in ("step_hbm_gbs", "dev_status", "cuda_graph"):
+    for k in ("step_hbm_gbs", "dev_status", "cuda_graph", "kernels"):
         if k in head:
             line[k] = head[k]
     line.update(extra)

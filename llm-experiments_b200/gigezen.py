@@ -23,6 +23,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Sequence, Tuple
 
+import numpy as np
 import torch
 
 from . import latent, moe
@@ -204,6 +205,30 @@ def prepare_weights(ctx: GPUContext, cfg: GigezenConfig, tensors: Dict[str, torc
                           final_norm=vec("final.norm", width), head=_b2(head))
 
 
+def random_tensors(ctx: GPUContext, config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
+    """Checkpoint tensors of a configuration drawn on the device (benchmarks): matrices N(0, 1 / fan_in), norms near identity."""
+    gen = torch.Generator(device=ctx.device).manual_seed(seed)
+    rnd = lambda shape, s: (torch.randn(shape, generator=gen, device=ctx.device) * s).to(torch.bfloat16)  # noqa: E731
+    mat = lambda out, inp: rnd((out, inp), inp ** -0.5)  # noqa: E731
+    width, t = config["width"], {}
+    t["embed"], t["head"], t["final.norm"] = rnd((config["vocab"], width), 1.0), mat(config["vocab"], width), rnd((width,), 0.1)
+    for i, entry in enumerate(config["layers"]):
+        p, m, mlp = f"l{i}.", entry["mixer"], entry.get("mlp")
+        t[p + "norm1"] = rnd((width,), 0.1)
+        t[p + "mix.q"] = mat(m["heads"] * (m["dim"] + m["rot_dim"]), width)
+        if m.get("kv_from") is None:
+            t[p + "mix.dkv"], t[p + "mix.dkv.norm"] = mat(m["kv_rank"] + m["rot_dim"], width), rnd((m["kv_rank"],), 0.1) + 1
+        t[p + "mix.uk"], t[p + "mix.uv"] = mat(m["heads"] * m["dim"], m["kv_rank"]), mat(m["heads"] * m["vdim"], m["kv_rank"])
+        t[p + "mix.o"] = mat(width, m["heads"] * m["vdim"])
+        blocks = [] if mlp is None else [(p + "mlp.", mlp["ff"])] if mlp["kind"] == "dense" else \
+            [(f"{p}mlp.e{e}.", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])]
+        for name, ff in blocks:
+            t[name + "gate"], t[name + "up"], t[name + "down"] = mat(ff, width), mat(ff, width), mat(width, ff)
+        if mlp is not None and mlp["kind"] == "moe":
+            t[p + "mlp.router"] = mat(mlp["router"]["experts"], width)
+    return t
+
+
 # ---------------------------------------------------------------------------------------------------------------
 # state
 # ---------------------------------------------------------------------------------------------------------------
@@ -234,10 +259,11 @@ class GigezenState:
         return self.owned[layer if src is None else src]
 
     def rows(self, name: str, rows: int, cols: int, dtype: torch.dtype) -> GPUBuffer2D:
-        """The first ``rows`` rows of a scratch buffer that grows on demand."""
+        """The first ``rows`` rows of a scratch buffer that grows on demand.  It starts at zero: padding columns that nothing
+        writes are multiplied with zero weights and must be numbers."""
         t = self.scratch.get(name)
         if t is None or t.shape[0] < rows or t.shape[1] != cols:
-            t = torch.empty((rows, cols), dtype=dtype, device=self.seq_lens.device)
+            t = torch.zeros((rows, cols), dtype=dtype, device=self.seq_lens.device)
             self.scratch[name] = t
         return GPUBuffer2D(buffer=t[:rows], shape=(rows, cols), size=rows * cols)
 
@@ -409,27 +435,28 @@ def forward(ctx: GPUContext, state: GigezenState, entries: Sequence[Tuple[int, S
     short = [len(t) <= SHORT_ENTRY or not state.prompt_form for _, t, _ in entries]
     order = sorted(range(len(entries)), key=lambda j: not short[j])  # stable: short entries first
     ids, slots, pos, first_row, spans, lens = [], [], [], {}, [], list(state.lengths)
-    n_single, span = 0, 1
+    T, n_single, span = 0, 0, 1
     for j in order:
         slot, tokens, _ = entries[j]
-        first_row[j] = len(ids)
+        first_row[j] = T
         start, n = lens[slot], len(tokens)
         if short[j]:
             n_single += n
             span = max(span, start + n)
         else:
-            spans.append((len(ids), n, slot, start))
-        ids += [int(t) for t in tokens]
-        slots += [slot] * n
-        pos += range(start, start + n)
+            spans.append((T, n, slot, start))
+        ids.append(np.asarray(tokens, dtype=np.int32))
+        slots.append(np.full(n, slot, dtype=np.int32))
+        pos.append(np.arange(start, start + n, dtype=np.int32))
+        T += n
         lens[slot] = start + n
     want = [first_row[j] + int(p) for j in range(len(entries)) for p in entries[j][2]]
-    T, n_out = len(ids), len(want)
+    n_out = len(want)
     windows = sorted({lc.attention.window for lc in state.cfg.layers}) if spans else []
     plans = {win: PromptPlan.build(spans, win, state.max_seq_len) for win in windows}
     # one upload per step: ids, sequences, positions, wanted rows, lengths behind the step, prompt tables
-    parts = [ids, slots, pos, want, lens] + [plans[win].rows() for win in windows]
-    host = torch.tensor([v for part in parts for v in part], dtype=torch.int32).pin_memory()
+    parts = [np.concatenate(ids), np.concatenate(slots), np.concatenate(pos), want, lens] + [plans[win].rows() for win in windows]
+    host = torch.from_numpy(np.concatenate([np.asarray(part, dtype=np.int32) for part in parts])).pin_memory()
     pieces = list(host.to(ctx.device, non_blocking=True).split([len(part) for part in parts]))
     for win, table in zip(windows, pieces[5:]):
         plans[win].table = table
