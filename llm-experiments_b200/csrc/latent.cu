@@ -13,12 +13,42 @@ namespace {
 constexpr int kAppendThreads = 256;
 constexpr int kMaxRot = 512;
 
+// Floats narrowed to one 16-byte piece of the storage type.
+__device__ __forceinline__ uint4 narrow(const float (&f)[4]) {
+    return make_uint4(__float_as_uint(f[0]), __float_as_uint(f[1]), __float_as_uint(f[2]), __float_as_uint(f[3]));
+}
+__device__ __forceinline__ uint4 narrow(const float (&f)[8]) {
+    uint32_t w[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+        w[e] = static_cast<uint32_t>(__bfloat16_as_ushort(__float2bfloat16_rn(f[2 * e]))) |
+               static_cast<uint32_t>(__bfloat16_as_ushort(__float2bfloat16_rn(f[2 * e + 1]))) << 16;
+    return make_uint4(w[0], w[1], w[2], w[3]);
+}
+
+// kPerChunk pairs of elements turned in place: (u, v) -> (u cos - v sin, v cos + u sin).
+template <typename T>
+__device__ __forceinline__ void rotate_pieces(uint4* pu, uint4* pv, const float* cs, const float* sn) {
+    constexpr int kC = Elt<T>::kPerChunk;
+    float u[kC], v[kC], a[kC], b[kC];
+    Elt<T>::widen(*pu, u);
+    Elt<T>::widen(*pv, v);
+#pragma unroll
+    for (int e = 0; e < kC; ++e) {
+        a[e] = u[e] * cs[e] - v[e] * sn[e];
+        b[e] = v[e] * cs[e] + u[e] * sn[e];
+    }
+    *pu = narrow(a);
+    *pv = narrow(b);
+}
+
+// vec: every head's rotated part, row and half of the rotated elements is made of whole 16-byte pieces.
 template <typename T>
 __global__ void __launch_bounds__(kAppendThreads)
 latent_append_kernel(T* y, int64_t ld_y, int H, int dim, int rot, int rot_dims, const float* inv_freq,
                      int down_col, int kv_rank, const float* w_norm, float eps, T* key_cache,
                      T* latent_cache, const int32_t* row_slot, const int32_t* row_pos,
-                     int n_slots, int T_max, int32_t* dev_status) {
+                     int n_slots, int T_max, int32_t* dev_status, bool vec) {
     __shared__ float cs[kMaxRot / 2], sn[kMaxRot / 2], part[kAppendThreads / 32];
     grid_launch_dependents();
     if (threadIdx.x == 0) grid_dependency_wait();
@@ -42,12 +72,22 @@ latent_append_kernel(T* y, int64_t ld_y, int H, int dim, int rot, int rot_dims, 
         if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = sum;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < H * half; i += kAppendThreads) {
-        const int h = i / half, j = i % half;
-        T* q = row + h * (dim + rot) + dim;
-        const float u = Elt<T>::to_float(q[j]), v = Elt<T>::to_float(q[j + half]);
-        q[j] = Elt<T>::from_float(u * cs[j] - v * sn[j]);
-        q[j + half] = Elt<T>::from_float(v * cs[j] + u * sn[j]);
+    constexpr int kC = Elt<T>::kPerChunk;
+    if (vec) {  // 16-byte pieces: kC pairs at a time
+        const int pieces = half / kC;
+        for (int i = threadIdx.x; i < H * pieces; i += kAppendThreads) {
+            const int h = i / pieces, j = i % pieces;
+            uint4* q = reinterpret_cast<uint4*>(row + h * (dim + rot) + dim);
+            rotate_pieces<T>(q + j, q + j + pieces, cs + j * kC, sn + j * kC);
+        }
+    } else {
+        for (int i = threadIdx.x; i < H * half; i += kAppendThreads) {
+            const int h = i / half, j = i % half;
+            T* q = row + h * (dim + rot) + dim;
+            const float u = Elt<T>::to_float(q[j]), v = Elt<T>::to_float(q[j + half]);
+            q[j] = Elt<T>::from_float(u * cs[j] - v * sn[j]);
+            q[j + half] = Elt<T>::from_float(v * cs[j] + u * sn[j]);
+        }
     }
     if (latent_cache == nullptr) return;
     sum = 0.f;
@@ -169,16 +209,18 @@ extern "C" int b2kv_latent_append(void* y, int64_t ld_y, int H, int dim, int rot
     if (rot_dims > kMaxRot) return B2KV_ERR_UNSUPPORTED;
     if ((key_cache == nullptr) != (latent_cache == nullptr)) return B2KV_ERR_BAD_ARG;
     if (latent_cache && (!w_norm || kv_rank <= 0 || down_col < 0 || ld_y < down_col + kv_rank + rot)) return B2KV_ERR_BAD_ARG;
+    const int per = 16 / elt_bytes(dtype);
+    const bool vec = aligned16(y) && ld_y % per == 0 && dim % per == 0 && rot % per == 0 && (rot_dims / 2) % per == 0;
     OverlapLaunch launch(rows, kAppendThreads, 0, stream);
     if (dtype == B2KV_DTYPE_F32)
         B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, latent_append_kernel<float>, static_cast<float*>(y), ld_y, H, dim, rot,
                                          rot_dims, inv_freq, down_col, kv_rank, w_norm, eps, static_cast<float*>(key_cache),
-                                         static_cast<float*>(latent_cache), row_slot, row_pos, n_slots, T_max, dev_status));
+                                         static_cast<float*>(latent_cache), row_slot, row_pos, n_slots, T_max, dev_status, vec));
     else
         B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, latent_append_kernel<__nv_bfloat16>, static_cast<__nv_bfloat16*>(y), ld_y,
                                          H, dim, rot, rot_dims, inv_freq, down_col, kv_rank, w_norm, eps,
                                          static_cast<__nv_bfloat16*>(key_cache), static_cast<__nv_bfloat16*>(latent_cache),
-                                         row_slot, row_pos, n_slots, T_max, dev_status));
+                                         row_slot, row_pos, n_slots, T_max, dev_status, vec));
     return B2KV_OK;
 }
 

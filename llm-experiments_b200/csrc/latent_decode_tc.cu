@@ -7,13 +7,17 @@
 //   S^T[key, head]     = latent[key, :] q_latent[head, :] + key part[key, :] q_rot[head, :]      A K-major
 //   O^T[element, head] += latent[:, element]^T P[key, head]                                       the same tile, A MN-major
 //
-//   * one CTA per (row, group of up to 64 heads, share of the row's window).  A tile is 128 keys: pairs of 64-element chunks
-//     of the latent rows and one chunk of the rotated key part, copied with TMA (128-byte swizzle) into a ring of pairs, so
-//     that the next tile's first pairs arrive while this one is still in use;
-//   * warp 4 copies, warp 5 issues tcgen05.mma from one thread, warps 0-3 are the softmax: thread = key = TMEM lane, one column
-//     per head.  Column maxima take one integer warp reduction per head and an exchange through shared memory; sums stay in
-//     registers per key until the end; P goes to shared memory as the K-major operand of the second product; O stays in tensor
-//     memory and is rescaled only when a head's maximum has grown by more than 2^8;
+//   * one CTA per (row, group of up to 64 heads, share of the row's window).  A tile is 64 keys, so that two and a half tiles
+//     of 512 + 64 elements fit shared memory: pairs of 64-element chunks of the latent rows, copied with TMA (128-byte swizzle)
+//     into a ring of pairs, and a chunk of the rotated key part in a ring of two.  An MMA has 128 rows all the same: the upper
+//     64 rows of S^T are made from whatever lies behind a chunk in shared memory, and nobody looks at them (64-row tiles of
+//     128-row MMAs waste tensor time that is not the limit; 128-key tiles left no room for the next tile's copies, and every
+//     tile then paid a full memory latency);
+//   * warp 4 copies, warp 5 issues tcgen05.mma from one thread, in the order S(j + 1), O(j), so that the next tile's scores are
+//     made under this tile's softmax.  Warps 0-1 are the softmax: thread = key = TMEM lane, one column per head.  Column maxima
+//     take one integer warp reduction per head and an exchange through shared memory; sums stay in registers per key until the
+//     end; P goes to shared memory as the K-major operand of the second product; O stays in tensor memory and is rescaled (by
+//     warps 0-3) only when a head's maximum has grown by more than 2^8;
 //   * the shares of one row (few rows, long windows) leave fp32 partial results that a small kernel merges.
 //
 // No MMA is predicated; sizes that do not fill a chunk read as zero.  Every wait is bounded.
@@ -30,8 +34,8 @@ namespace latdec {
 
 using namespace tc;
 
-constexpr int kTile = 128;               // keys per tile
-constexpr int kChunkBytes = kTile * 128;  // 128 rows x 64 bf16
+constexpr int kTile = 64;                // keys per tile
+constexpr int kChunkBytes = kTile * 128;  // 64 rows x 64 bf16
 constexpr int kPairBytes = 2 * kChunkBytes;
 constexpr int kMaxPairs = 12;
 constexpr int kMaxHeads = 64;
@@ -43,13 +47,13 @@ constexpr float kNothingSeen = -1e30f;
 struct Shared {
     alignas(8) uint64_t q_full;
     uint64_t pair_full[kMaxPairs], pair_empty[kMaxPairs];
-    uint64_t rot_full, rot_empty;
-    uint64_t s_full, p_ready, o_done;
+    uint64_t rot_full[2], rot_empty[2];
+    uint64_t s_full[2], p_ready[2], o_done;
     uint32_t tmem_base;
     volatile int abort_flag;
     int need;
-    int warp_max[4][kMaxHeads];
-    float m[kMaxHeads], factor[kMaxHeads], sum[4][kMaxHeads];
+    int warp_max[2][kMaxHeads];
+    float m[kMaxHeads], factor[kMaxHeads], sum[2][kMaxHeads];
 };
 
 struct Params {
@@ -80,9 +84,9 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
     __shared__ Shared sm;
     uint8_t* const ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     uint8_t* const rot_tile = ring + p.ring_pairs * kPairBytes;
-    uint8_t* const q_tile = rot_tile + kChunkBytes;  // 2 * tile_pairs latent chunks, then the rotated one; kHn rows each
+    uint8_t* const q_tile = rot_tile + 2 * kChunkBytes;  // 2 * tile_pairs latent chunks, then the rotated one; kHn rows each
     constexpr int kQChunk = kHn * 128;
-    uint8_t* const p_tile = q_tile + (2 * p.tile_pairs + 1) * kQChunk;  // [2][kHn][64 keys]
+    uint8_t* const p_tile = q_tile + (2 * p.tile_pairs + 1) * kQChunk;  // two tiles of [kHn][64 keys]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int split = blockIdx.x % p.splits;
     const int h0 = blockIdx.x / p.splits % p.head_groups * kHn;
@@ -95,10 +99,12 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
             mbar_init(&sm.pair_full[s], 1);
             mbar_init(&sm.pair_empty[s], 1);
         }
-        mbar_init(&sm.rot_full, 1);
-        mbar_init(&sm.rot_empty, 1);
-        mbar_init(&sm.s_full, 1);
-        mbar_init(&sm.p_ready, 128);
+        for (int s = 0; s < 2; ++s) {
+            mbar_init(&sm.rot_full[s], 1);
+            mbar_init(&sm.rot_empty[s], 1);
+            mbar_init(&sm.s_full[s], 1);
+            mbar_init(&sm.p_ready[s], 128);
+        }
         mbar_init(&sm.o_done, 1);
         sm.abort_flag = 0;
         sm.need = 0;
@@ -123,7 +129,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
     const int first = split * share;
     const int n_tiles = max(0, min(share, all_tiles - first));
     if (!valid && threadIdx.x == 0) report_status(p.dev_status, B2KV_DEV_BAD_POSITION);
-    const uint32_t o_base = tmem + kHn;  // S in columns [0, kHn), O of pair g behind it
+    const uint32_t o_base = tmem + 2 * kHn;  // S of even and odd tiles in columns [0, 2 kHn), O of pair g behind them
 
     if (warp == 4) {
         // ------------------------------ TMA producer ------------------------------
@@ -136,10 +142,10 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
             uint32_t phase = 1;  // parity of the "empty" phase to wait for: the ring starts empty
             for (int j = 0; j < n_tiles && ok; ++j) {
                 const int row = slot * p.T_max + t0 + (first + j) * kTile;
-                ok = mbar_wait(&sm.rot_empty, (j & 1) ^ 1);
+                ok = mbar_wait(&sm.rot_empty[j & 1], ((j >> 1) & 1) ^ 1);
                 if (!ok) break;
-                mbar_arrive_expect_tx(&sm.rot_full, kChunkBytes);
-                tma_load_3d(rot_tile, &tm_key, &sm.rot_full, 0, 0, row);
+                mbar_arrive_expect_tx(&sm.rot_full[j & 1], kChunkBytes);
+                tma_load_3d(rot_tile + (j & 1) * kChunkBytes, &tm_key, &sm.rot_full[j & 1], 0, 0, row);
                 for (int g = 0; g < p.tile_pairs; ++g) {
                     ok = mbar_wait(&sm.pair_empty[slot_i], phase);
                     if (!ok) break;
@@ -162,49 +168,54 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
             const uint64_t d_q = smem_desc(smem_u32(q_tile), 16, 1024), d_p = smem_desc(smem_u32(p_tile), 16, 1024);
             constexpr uint32_t kPair16 = kPairBytes >> 4, kChunk16 = kChunkBytes >> 4, kQ16 = kQChunk >> 4;
             const uint64_t d_qr = d_q + static_cast<uint64_t>(2 * p.tile_pairs) * kQ16;
-            bool ok = mbar_wait(&sm.q_full, 0);
-            int slot_i = 0;
+            int slot_i = 0, done_i = 0;  // ring places of the next pair to multiply with the queries / with P
             uint32_t phase = 0;
-            for (int j = 0; j < n_tiles && ok; ++j) {
-                ok = mbar_wait(&sm.rot_full, j & 1);
-                if (!ok) break;
+            bool ok = mbar_wait(&sm.q_full, 0);
+            // scores of tile j
+            auto issue_s = [&](int j) {
+                if (!mbar_wait(&sm.rot_full[j & 1], (j >> 1) & 1)) return false;
                 tc_fence_after();
+                const uint32_t s_tmem = tmem + (j & 1) * kHn;
+                const uint64_t ar = d_rot + static_cast<uint64_t>(j & 1) * kChunk16;
 #pragma unroll
                 for (int kk = 0; kk < 4; ++kk)
-                    mma_ss(tmem, d_rot + static_cast<uint64_t>(2 * kk), d_qr + static_cast<uint64_t>(2 * kk), idesc_s, kk ? 1u : 0u);
-                mma_commit(&sm.rot_empty);
-                const int tile_slot = slot_i;
+                    mma_ss(s_tmem, ar + static_cast<uint64_t>(2 * kk), d_qr + static_cast<uint64_t>(2 * kk), idesc_s, kk ? 1u : 0u);
+                mma_commit(&sm.rot_empty[j & 1]);
                 for (int g = 0; g < p.tile_pairs; ++g) {
-                    ok = mbar_wait(&sm.pair_full[slot_i], phase);
-                    if (!ok) break;
+                    if (!mbar_wait(&sm.pair_full[slot_i], phase)) return false;
                     tc_fence_after();
                     const uint64_t a = d_lat_k + static_cast<uint64_t>(slot_i) * kPair16;
                     const uint64_t b = d_q + static_cast<uint64_t>(2 * g) * kQ16;
 #pragma unroll
                     for (int kk = 0; kk < 8; ++kk)
-                        mma_ss(tmem, a + static_cast<uint64_t>((kk >> 2) * kChunk16 + (kk & 3) * 2),
+                        mma_ss(s_tmem, a + static_cast<uint64_t>((kk >> 2) * kChunk16 + (kk & 3) * 2),
                                b + static_cast<uint64_t>((kk >> 2) * kQ16 + (kk & 3) * 2), idesc_s, 1u);
                     if (++slot_i == p.ring_pairs) slot_i = 0, phase ^= 1;
                 }
-                if (!ok) break;
-                mma_commit(&sm.s_full);
-                ok = mbar_wait(&sm.p_ready, j & 1);
+                mma_commit(&sm.s_full[j & 1]);
+                return true;
+            };
+            ok = ok && issue_s(0);
+            for (int j = 0; j < n_tiles && ok; ++j) {
+                // P(j - 1) has been waited for, so S(j - 1) has been read and its columns are free
+                if (j + 1 < n_tiles) ok = issue_s(j + 1);
+                ok = ok && mbar_wait(&sm.p_ready[j & 1], (j >> 1) & 1);
                 if (!ok) break;
                 tc_fence_after();
-                int s = tile_slot;
+                const uint64_t b = d_p + static_cast<uint64_t>(j & 1) * kQ16;
                 for (int g = 0; g < p.tile_pairs; ++g) {
-                    const uint64_t a = d_lat_mn + static_cast<uint64_t>(s) * kPair16;
+                    const uint64_t a = d_lat_mn + static_cast<uint64_t>(done_i) * kPair16;
                     const uint32_t o = o_base + g * kHn;
 #pragma unroll
-                    for (int kk = 0; kk < 8; ++kk)  // 16 keys: 2048 bytes of the tile, 32 bytes of P (next chunk after four)
-                        mma_ss(o, a + static_cast<uint64_t>((kk * 2048) >> 4),
-                               d_p + static_cast<uint64_t>((kk >> 2) * kQ16 + (kk & 3) * 2), idesc_o, (j | kk) ? 1u : 0u);
-                    mma_commit(&sm.pair_empty[s]);
-                    if (++s == p.ring_pairs) s = 0;
+                    for (int kk = 0; kk < 4; ++kk)  // 16 keys: 2048 bytes of the tile, 32 bytes of P
+                        mma_ss(o, a + static_cast<uint64_t>((kk * 2048) >> 4), b + static_cast<uint64_t>(2 * kk), idesc_o,
+                               (j | kk) ? 1u : 0u);
+                    mma_commit(&sm.pair_empty[done_i]);
+                    if (++done_i == p.ring_pairs) done_i = 0;
                 }
+                mma_commit(&sm.o_done);
             }
-            if (ok) mma_commit(&sm.o_done);
-            else sm.abort_flag = 1;
+            if (!ok) sm.abort_flag = 1;
         }
         __syncwarp();
     } else {
@@ -217,24 +228,27 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
         for (int h = 0; h < kHn; ++h) l[h] = 0.f;
         bool ok = true;
         for (int j = 0; j < n_tiles; ++j) {
-            ok = __all_sync(0xffffffffu, mbar_wait(&sm.s_full, j & 1));
+            ok = __all_sync(0xffffffffu, mbar_wait(&sm.s_full[j & 1], (j >> 1) & 1));
             if (!ok) break;
             tc_fence_after();
-            const bool seen = t0 + (first + j) * kTile + key <= pos;
             uint32_t r[kHn];
+            if (warp < kTile / 32) {
+                const bool seen = t0 + (first + j) * kTile + key <= pos;
 #pragma unroll
-            for (int cc = 0; cc < kHn / 16; ++cc) tmem_ld16(tmem + lane_base + cc * 16, *reinterpret_cast<uint32_t(*)[16]>(&r[cc * 16]));
-            tmem_wait_ld();
+                for (int cc = 0; cc < kHn / 16; ++cc)
+                    tmem_ld16(tmem + lane_base + (j & 1) * kHn + cc * 16, *reinterpret_cast<uint32_t(*)[16]>(&r[cc * 16]));
+                tmem_wait_ld();
 #pragma unroll
-            for (int h = 0; h < kHn; ++h) {
-                r[h] = seen ? r[h] : 0xff800000u;
-                const int mx = __reduce_max_sync(0xffffffffu, ordered(__uint_as_float(r[h])));
-                if (lane == (h & 31)) sm.warp_max[warp][h] = mx;
+                for (int h = 0; h < kHn; ++h) {
+                    r[h] = seen ? r[h] : 0xff800000u;
+                    const int mx = __reduce_max_sync(0xffffffffu, ordered(__uint_as_float(r[h])));
+                    if (lane == (h & 31)) sm.warp_max[warp][h] = mx;
+                }
             }
             named_barrier_sync<128>(1);
             if (threadIdx.x < kHn) {
                 const int h = threadIdx.x;
-                const float mx = unordered(max(max(sm.warp_max[0][h], sm.warp_max[1][h]), max(sm.warp_max[2][h], sm.warp_max[3][h]))) * c;
+                const float mx = unordered(max(sm.warp_max[0][h], sm.warp_max[1][h])) * c;
                 float m = j == 0 ? fmaxf(mx, kNothingSeen) : sm.m[h], f = 1.f;
                 if (mx > m + kRescaleThreshold) {
                     f = ex2(m - mx);
@@ -246,15 +260,20 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
             }
             named_barrier_sync<128>(1);
             const bool need = *reinterpret_cast<volatile int*>(&sm.need) == j + 1;
-            // P of the tile before has been read: its product was issued before this tile's scores
+            // P of the tile before last has been read: its product was issued before this tile's scores
+            if (warp < kTile / 32) {
+                uint8_t* const p_row = p_tile + (j & 1) * kQChunk + (key & 7) * 2;
 #pragma unroll
-            for (int h = 0; h < kHn; ++h) {
-                const float w = ex2(fmaf(__uint_as_float(r[h]), c, -sm.m[h]));
-                l[h] = l[h] * sm.factor[h] + w;
-                uint8_t* dst = p_tile + (key >> 6) * kQChunk + h * 128 + ((((key & 63) >> 3) ^ (h & 7)) << 4) + (key & 7) * 2;
-                *reinterpret_cast<__nv_bfloat16*>(dst) = __float2bfloat16_rn(w);
+                for (int h = 0; h < kHn; ++h) {
+                    const float w = ex2(fmaf(__uint_as_float(r[h]), c, -sm.m[h]));
+                    l[h] = l[h] * sm.factor[h] + w;
+                    *reinterpret_cast<__nv_bfloat16*>(p_row + h * 128 + (((key >> 3) ^ (h & 7)) << 4)) = __float2bfloat16_rn(w);
+                }
             }
-            if (need) {  // (uniform) bring O down to the new reference maxima
+            if (need && j > 0) {  // (uniform) bring O down to the new reference maxima, once the product before has gone into it
+                ok = __all_sync(0xffffffffu, mbar_wait(&sm.o_done, (j - 1) & 1));
+                if (!ok) break;
+                tc_fence_after();
 #pragma unroll 1
                 for (int g = 0; g < p.tile_pairs; ++g) {
 #pragma unroll
@@ -272,9 +291,11 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
             }
             fence_proxy_async_smem();  // P was written with ordinary stores and is read by the tensor core
             tc_fence_before();
-            mbar_arrive(&sm.p_ready);
+            mbar_arrive(&sm.p_ready[j & 1]);
         }
-        if (n_tiles > 0 && ok) ok = __all_sync(0xffffffffu, mbar_wait(&sm.o_done, 0));
+        // (a parity wait cannot tell a phase from the one two before: the last scores waited for cover all products but two)
+        if (n_tiles > 1 && ok) ok = __all_sync(0xffffffffu, mbar_wait(&sm.o_done, (n_tiles - 2) & 1));
+        if (n_tiles > 0 && ok) ok = __all_sync(0xffffffffu, mbar_wait(&sm.o_done, (n_tiles - 1) & 1));
         if (ok) {
             tc_fence_after();
             // sums over the keys: inside the warps, then over the warps
@@ -282,7 +303,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
             for (int h = 0; h < kHn; ++h) {
 #pragma unroll
                 for (int off = 16; off > 0; off >>= 1) l[h] += __shfl_xor_sync(0xffffffffu, l[h], off);
-                if (lane == (h & 31)) sm.sum[warp][h] = l[h];
+                if (lane == (h & 31) && warp < kTile / 32) sm.sum[warp][h] = l[h];
             }
             named_barrier_sync<128>(1);
             const int heads = min(kHn, p.H - h0);
@@ -291,7 +312,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
             if (part != nullptr && threadIdx.x < heads) {
                 const int h = threadIdx.x;
                 part[h * stride + p.kv_rank] = n_tiles > 0 ? sm.m[h] : kNothingSeen;
-                part[h * stride + p.kv_rank + 1] = (sm.sum[0][h] + sm.sum[1][h]) + (sm.sum[2][h] + sm.sum[3][h]);
+                part[h * stride + p.kv_rank + 1] = sm.sum[0][h] + sm.sum[1][h];
             }
             if (n_tiles > 0) {
                 __nv_bfloat16* out = p.out + (static_cast<int64_t>(i) * p.H + h0) * p.kv_rank;
@@ -313,7 +334,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_ql, const __grid_
                                 part[h * stride + e] = v;
                             else
                                 out[static_cast<int64_t>(h) * p.kv_rank + e] =
-                                    __float2bfloat16_rn(v / ((sm.sum[0][h] + sm.sum[1][h]) + (sm.sum[2][h] + sm.sum[3][h])));
+                                    __float2bfloat16_rn(v / (sm.sum[0][h] + sm.sum[1][h]));
                         }
                     }
                 }
@@ -383,12 +404,12 @@ static bool make_map(CUtensorMap* map, const void* base, int width, int heads, i
 
 static int head_columns(int H) { return H <= 16 ? 16 : (H <= 32 ? 32 : 64); }
 
-// Shares per row: about one CTA per SM, each with at least two tiles where the window has them.
+// Shares per row: about one CTA per SM, each with at least four tiles where the window has them.
 static int choose_splits(int rows, int H, int span) {
     const int groups = (H + kMaxHeads - 1) / kMaxHeads;
     const int tiles = (span + kTile - 1) / kTile;
     const int fill = std::max(1, device_sm_count() / std::max(1, rows * groups));
-    return std::max(1, std::min(std::min(fill, kMaxSplits), (tiles + 1) / 2));
+    return std::max(1, std::min(std::min(fill, kMaxSplits), (tiles + 3) / 4));
 }
 
 template <int kHn>
@@ -421,11 +442,11 @@ int latent_decode_tc(const LatentDecodeArgs& a, void* workspace, size_t workspac
     if (static_cast<int64_t>(a.n_slots) * a.T_max > 0x7fffffffLL - 256) return B2KV_ERR_UNSUPPORTED;
     const int tile_pairs = (a.kv_rank + 127) / 128;
     auto fixed_bytes = [&](int hn) {
-        return kChunkBytes + (2 * tile_pairs + 1) * hn * 128 + 2 * hn * 128 + 1024 + static_cast<int>(sizeof(Shared));
+        return 2 * kChunkBytes + (2 * tile_pairs + 1) * hn * 128 + 2 * hn * 128 + 1024 + static_cast<int>(sizeof(Shared));
     };
     int Hn = head_columns(a.H);
     // 64 heads beside a wide latent do not fit one SM: two groups of 32 then read the same rows, the second out of L2
-    while (Hn > 16 && (kSmemLimit - fixed_bytes(Hn)) / kPairBytes < tile_pairs) Hn /= 2;
+    while (Hn > 16 && (kSmemLimit - fixed_bytes(Hn)) / kPairBytes < 2 * tile_pairs) Hn /= 2;
     Params p{};
     p.row_slot = a.row_slot;
     p.row_pos = a.row_pos;
@@ -444,10 +465,10 @@ int latent_decode_tc(const LatentDecodeArgs& a, void* workspace, size_t workspac
         return B2KV_ERR_WORKSPACE;
     p.tile_pairs = tile_pairs;
     p.tmem_cols = 32;
-    while (p.tmem_cols < (p.tile_pairs + 1) * Hn) p.tmem_cols *= 2;
+    while (p.tmem_cols < (p.tile_pairs + 2) * Hn) p.tmem_cols *= 2;
     const int fixed = fixed_bytes(Hn);
     p.ring_pairs = std::min(std::min(kMaxPairs, 3 * p.tile_pairs), (kSmemLimit - fixed) / kPairBytes);
-    if (p.ring_pairs < p.tile_pairs) return B2KV_ERR_UNSUPPORTED;
+    if (p.ring_pairs < 2 * p.tile_pairs) return B2KV_ERR_UNSUPPORTED;
     const size_t smem = static_cast<size_t>(p.ring_pairs) * kPairBytes + fixed - sizeof(Shared);
     const int64_t cache_rows = static_cast<int64_t>(a.n_slots) * a.T_max;
     CUtensorMap m[4];

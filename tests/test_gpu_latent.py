@@ -41,7 +41,7 @@ def run(pkg, ctx, fn, *a, **kw):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF])
-@pytest.mark.parametrize("H,dim,rot,rank,base", [(3, 8, 4, 10, 500.0), (6, 48, 24, 72, 10000.0), (2, 128, 64, 512, 1e6)])
+@pytest.mark.parametrize("H,dim,rot,rank,base", [(3, 8, 4, 10, 500.0), (6, 48, 24, 72, 10000.0), (2, 128, 64, 512, 1e6), (5, 48, 16, 72, 1e4)])
 def test_append_norms_rotates_and_stores(pkg, dtype, H, dim, rot, rank, base):
     """Rows of several sequences at scattered positions; every other cache row keeps its value."""
     from llm_experiments_b200 import latent
@@ -51,7 +51,7 @@ def test_append_norms_rotates_and_stores(pkg, dtype, H, dim, rot, rank, base):
     cache, key, lat = make_cache(pkg, ctx, 3, 4096, rot, rank, dtype)
     key.fill_(3.0), lat.fill_(3.0)
     q_cols = H * (dim + rot)
-    y = rnd((5, q_cols + rank + rot + 7), dtype, 1)
+    y = rnd((5, q_cols + rank + rot + (7 if dim == 8 else 8)), dtype, 1)
     before = to_f32(y).astype(np.float64)
     w = torch.randn(rank, device="cuda") + 1
     inv = torch.tensor([base ** (-2.0 * j / rot) for j in range(rot // 2)], dtype=F32, device="cuda")
