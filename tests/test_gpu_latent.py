@@ -101,7 +101,7 @@ def single_rows(q_lat, q, lat, key, slot, pos, shape):
 
 
 CASES = [  # heads, dim, rot, kv_rank, window, positions
-    (6, 8, 16, 64, 40, (0, 1, 38, 39, 40, 41, 300)), (3, 24, 8, 40, 1, (0, 5, 127, 128, 129)),
+    (7, 8, 16, 56, 45, (0, 1, 43, 44, 45, 46, 300)), (3, 24, 8, 40, 1, (0, 5, 127, 128, 129)),
     (16, 16, 64, 512, 129, (0, 127, 128, 129, 900)), (32, 8, 32, 256, 0, (500, 3)), (50, 8, 64, 512, 200, (700, 10)),
     (70, 8, 24, 136, 0, (383, 384)), (5, 8, 16, 128, 0, (1000,)), (16, 8, 64, 512, 0, tuple(range(250, 250 + 40)))]
 
@@ -176,7 +176,7 @@ def test_fp32_single_rows(pkg):
     torch.testing.assert_close(out.double().cpu(), single_rows(ql, q, lat, key, slot, pos, shape), rtol=1e-5, atol=1e-5)
 
 
-@pytest.mark.parametrize("H,dim,rot,vdim", [(3, 128, 64, 128), (2, 64, 32, 64), (3, 128, 64, 64), (2, 64, 16, 128), (3, 48, 24, 40),
+@pytest.mark.parametrize("H,dim,rot,vdim", [(3, 128, 64, 128), (2, 64, 40, 56), (3, 128, 64, 64), (2, 64, 16, 128), (3, 48, 24, 40),
                                             (2, 96, 64, 80)])
 @pytest.mark.parametrize("window", [0, 1, 17, 128, 300])
 def test_prompt_portions(pkg, H, dim, rot, vdim, window):

@@ -45,7 +45,7 @@ def run(pkg, ctx, *a, **kw):
 
 @pytest.mark.parametrize("path,dtype,rows,K,cols", [
     (SIMT, torch.float32, 5, 37, (30, 7)), (SIMT, torch.bfloat16, 70, 100, (64, 33)),
-    (ROWS, torch.bfloat16, 1, 192, (64, 24)), (ROWS, torch.bfloat16, 3, 72, (32, 40)),
+    (ROWS, torch.bfloat16, 1, 176, (64, 24)), (ROWS, torch.bfloat16, 3, 72, (32, 40)),
     (ROWS, torch.bfloat16, 64, 1000, (96, 200)), (ROWS, torch.bfloat16, 128, 4096, (256, 256)),
     (TILED, torch.bfloat16, 129, 64, (32, 16)), (TILED, torch.bfloat16, 300, 200, (320, 72)),
     (TILED, torch.bfloat16, 1000, 520, (64, 704))])
@@ -74,7 +74,7 @@ def test_store_and_fp32_segments(pkg, path, dtype, rows, K, cols):
 @pytest.mark.parametrize("kind", ["SEG_GLU_SILU", "SEG_GLU_CLAMP"])
 @pytest.mark.parametrize("path,dtype,rows,K,ff", [
     (SIMT, torch.float32, 9, 40, 21), (ROWS, torch.bfloat16, 2, 96, 48), (ROWS, torch.bfloat16, 33, 2048, 64),
-    (ROWS, torch.bfloat16, 100, 256, 400), (TILED, torch.bfloat16, 200, 256, 208), (TILED, torch.bfloat16, 600, 192, 384)])
+    (ROWS, torch.bfloat16, 100, 256, 400), (TILED, torch.bfloat16, 200, 256, 208), (TILED, torch.bfloat16, 600, 208, 352)])
 def test_gated_segments(pkg, kind, path, dtype, rows, K, ff):
     from llm_experiments_b200 import projection as proj
 
@@ -92,7 +92,7 @@ def test_gated_segments(pkg, kind, path, dtype, rows, K, ff):
 
 
 @pytest.mark.parametrize("path,dtype,rows,heads,k,n,gap", [
-    (SIMT, torch.float32, 3, 5, 12, 20, 7), (ROWS, torch.bfloat16, 4, 6, 64, 64, 32), (ROWS, torch.bfloat16, 17, 3, 40, 136, 24),
+    (SIMT, torch.float32, 3, 5, 12, 20, 7), (ROWS, torch.bfloat16, 4, 7, 56, 72, 40), (ROWS, torch.bfloat16, 17, 3, 40, 136, 24),
     (ROWS, torch.bfloat16, 64, 16, 128, 512, 64), (0, torch.bfloat16, 300, 4, 64, 96, 16)])
 def test_per_head_products(pkg, path, dtype, rows, heads, k, n, gap):
     """Head h multiplies its own columns of x with its own matrix; what lies between the heads' columns is not touched, even
@@ -124,7 +124,7 @@ def test_per_head_columns_of_one_matrix(pkg):
 
 
 @pytest.mark.parametrize("path,dtype,counts,K,n,glu_kind", [
-    (SIMT, torch.float32, (3, 0, 5, 1), 20, 24, False), (ROWS, torch.bfloat16, (3, 0, 17, 1, 0), 192, 64, True),
+    (SIMT, torch.float32, (3, 0, 5, 1), 20, 24, False), (ROWS, torch.bfloat16, (3, 0, 17, 1, 0), 176, 96, True),
     (ROWS, torch.bfloat16, (0, 128, 1), 1408, 264, False), (TILED, torch.bfloat16, (0, 300, 1, 128, 0, 257, 129), 64, 328, False),
     (TILED, torch.bfloat16, (700, 513, 0), 256, 272, True)])
 def test_rows_grouped_by_expert(pkg, path, dtype, counts, K, n, glu_kind):
