@@ -33,13 +33,12 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = u;
 }
 
-// One CTA per row; a row of up to 16384 elements stays in registers between the two passes.
-template <typename T>
+// One CTA per row; a row of up to 1024 * kKeep elements stays in registers between the two passes.
+template <typename T, int kKeep>
 __global__ void __launch_bounds__(kThreads) rmsnorm_kernel(const float* x, int64_t ld_x,
                                                            const int32_t* row_index, const float* w,
                                                            float w_offset, T* out, int64_t ld_out, int size,
                                                            float eps, bool vec) {
-    constexpr int kKeep = 16;
     __shared__ float part[kThreads / 32];
     grid_launch_dependents();
     if (threadIdx.x == 0) grid_dependency_wait();
@@ -87,6 +86,16 @@ __global__ void __launch_bounds__(kThreads) rmsnorm_kernel(const float* x, int64
     }
 }
 
+template <typename T>
+int launch_rmsnorm(const float* x, int64_t ld_x, const int32_t* row_index, const float* w, float w_offset, T* out, int64_t ld_out,
+                   int rows, int size, float eps, bool vec, void* stream) {
+    // few registers per thread for rows of usual width: more CTAs per SM hide each other's two passes
+    auto kernel = size <= 4096 ? rmsnorm_kernel<T, 4> : (size <= 8192 ? rmsnorm_kernel<T, 8> : rmsnorm_kernel<T, 16>);
+    OverlapLaunch launch(rows, kThreads, 0, stream);
+    B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, kernel, x, ld_x, row_index, w, w_offset, out, ld_out, size, eps, vec));
+    return B2KV_OK;
+}
+
 }  // namespace
 }  // namespace b2kv
 
@@ -111,12 +120,6 @@ extern "C" int b2kv_rmsnorm(const float* x, int64_t ld_x, const int32_t* row_ind
     if (elt_bytes(dtype) == 0) return B2KV_ERR_UNSUPPORTED;
     if (!x || !w || !out || rows <= 0 || size <= 0 || ld_x < size || ld_out < size) return B2KV_ERR_BAD_ARG;
     const bool vec = size % 4 == 0 && ld_x % 4 == 0 && ld_out % 4 == 0 && size <= 16384 && aligned16(x) && aligned16(w) && aligned16(out);
-    OverlapLaunch launch(rows, kThreads, 0, stream);
-    if (dtype == B2KV_DTYPE_F32)
-        B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, rmsnorm_kernel<float>, x, ld_x, row_index, w, w_offset,
-                                         static_cast<float*>(out), ld_out, size, eps, vec));
-    else
-        B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, rmsnorm_kernel<__nv_bfloat16>, x, ld_x, row_index, w, w_offset,
-                                         static_cast<__nv_bfloat16*>(out), ld_out, size, eps, vec));
-    return B2KV_OK;
+    if (dtype == B2KV_DTYPE_F32) return launch_rmsnorm(x, ld_x, row_index, w, w_offset, static_cast<float*>(out), ld_out, rows, size, eps, vec, stream);
+    return launch_rmsnorm(x, ld_x, row_index, w, w_offset, static_cast<__nv_bfloat16*>(out), ld_out, rows, size, eps, vec, stream);
 }
