@@ -370,22 +370,33 @@ int b2kv_matmul(const void* a, const void* w, const void* bias, const void* resi
  * storage type of activations and weights; norms, rotations, scores, routers and the residual are computed in 32-bit.
  */
 
-/* out[i, :] = table[ids[i], :] in fp32 (the start of a 32-bit residual stream; no position is added).  A token id outside
- * the table is clamped and recorded in dev_status. */
-int b2kv_embed_rows(const void* table, const int32_t* ids, float* out, int rows, int dim, int vocab, int dtype,
-                    int32_t* dev_status, void* stream);
+/* out[i, :] = table[ids[i], :] * scale in fp32 (the start of a 32-bit residual stream; no position is added); with `copy`
+ * ([rows, dim] of `dtype`, or NULL) the same rows in the storage type as well.  A token id outside the table is clamped and
+ * recorded in dev_status. */
+int b2kv_embed_rows(const void* table, const int32_t* ids, float* out, void* copy, float scale, int rows, int dim, int vocab,
+                    int dtype, int32_t* dev_status, void* stream);
 
 /* out[i, :] = x[r, :] / sqrt(mean(x[r, :]^2) + eps) * (w + w_offset), r = row_index ? row_index[i] : i; x and w fp32, out
  * of `dtype`.  w_offset = 1 is the form whose weights are stored around zero. */
 int b2kv_rmsnorm(const float* x, int64_t ld_x, const int32_t* row_index, const float* w, float w_offset, void* out,
                  int64_t ld_out, int rows, int size, float eps, int dtype, void* stream);
 
+/* Layer norm of fp32 rows: v = (y[r, :] - mean) / sqrt(variance + eps) * w + b, r = row_index ? row_index[i] : i, the variance
+ * being the mean of the squared deviations.  With x (fp32) the rows are added to it: x[i, :] += v, the residual of a block
+ * whose norm sits behind the sublayer; without x they are only stored.  out (of `dtype`, may be NULL when x is given) gets
+ * the new x[i, :], or v.  y, x, w and b are fp32. */
+int b2kv_layernorm_rows(const float* y, int64_t ld_y, const int32_t* row_index, const float* w, const float* b, float* x,
+                        int64_t ld_x, void* out, int64_t ld_out, int rows, int size, float eps, int dtype, void* stream);
+
 /*
- * out = x @ w per group, with the output columns cut into up to three segments that go to places of their own:
+ * out = x @ w (+ bias) per group, with the output columns cut into up to three segments that go to places of their own:
  *   B2KV_SEG_STORE      the product, in the storage type
  *   B2KV_SEG_F32        the product (+ residual), fp32: the residual stream, router scores, logits
  *   B2KV_SEG_GLU_SILU   columns come in pairs (gate, up): silu(gate) * up, half as many output columns
  *   B2KV_SEG_GLU_CLAMP  pairs (gate, up): g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1)
+ *   B2KV_SEG_RELU2      max(product, 0)^2, in the storage type
+ *   B2KV_SEG_SOFTCAP    limit * tanh(product / limit), fp32
+ * bias is fp32 [N] (NULL: none; products without groups only).
  * x is [rows, K] with row pitch ld_x; w is [K, N] row-major with row pitch ld_w.  Group g (0 <= g < groups) reads
  * x + g * group_x and w + g * group_w and writes seg.out + g * seg.group: the heads of a per-head product.  With group_rows
  * (device, groups + 1 row offsets) group g instead owns rows group_rows[g] .. group_rows[g + 1] - 1 of x and of the outputs:
@@ -399,6 +410,8 @@ int b2kv_rmsnorm(const float* x, int64_t ld_x, const int32_t* row_index, const f
 #define B2KV_SEG_F32 1
 #define B2KV_SEG_GLU_SILU 2
 #define B2KV_SEG_GLU_CLAMP 3
+#define B2KV_SEG_RELU2 4
+#define B2KV_SEG_SOFTCAP 5
 #define B2KV_MAX_SEGMENTS 3
 typedef struct b2kv_segment {
     void* out;
@@ -408,7 +421,8 @@ typedef struct b2kv_segment {
 typedef struct b2kv_linear_args {
     const void* x;
     const void* w;
-    const float* residual; /* added to fp32 segments (may be the output itself), or NULL */
+    const float* residual; /* added to B2KV_SEG_F32 segments (may be the output itself), or NULL */
+    const float* bias;
     const int32_t* group_rows;
     int64_t ld_x, group_x, ld_w, group_w, ld_residual;
     b2kv_segment seg[B2KV_MAX_SEGMENTS];
@@ -465,6 +479,77 @@ int b2kv_latent_prefill(const void* q, int64_t ld_q, const void* keys, const voi
                         int64_t cache_rows, void* out, int64_t ld_out, const b2kv_prompt_segment* segments, int n_segments,
                         int n_blocks, int rows, int kv_rows, int H, int dim, int rot, int vdim, int window, float scale, int dtype,
                         int32_t* dev_status, void* stream);
+
+/*
+ * Grouped-query attention with an optional distance bias, on caches [sequences * T_max, G * dim] (keys) and
+ * [sequences * T_max, G * vdim] (values).  Query head h reads key / value head h / (H / G).  b2kv_gqa_append, per row i of y
+ * ([q: H * dim | k: G * dim | v: G * vdim], or the queries alone when k_cache is NULL) at position p = row_pos[i] of sequence
+ * row_slot[i] (row_slot NULL: sequence i):
+ *   - q, and k, are RMS-normed over all their heads at once with the factors q_norm [H * dim], k_norm [G * dim] (NULL: not
+ *     normed) and eps; q is multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) (temp_every <= 0: by one) and
+ *     left in place;
+ *   - k and v are stored at their place in the caches.
+ * A position outside [0, T_max) is skipped and recorded in dev_status.
+ */
+int b2kv_gqa_append(void* y, int64_t ld_y, int H, int G, int dim, int vdim, const float* q_norm, const float* k_norm, float eps,
+                    float temp_coef, int temp_every, void* k_cache, void* v_cache, const int32_t* row_slot,
+                    const int32_t* row_pos, int n_slots, int T_max, int rows, int dtype, int32_t* dev_status, void* stream);
+
+/*
+ * Attention of single query rows (decoding, short portions) over such caches: per row i and head h
+ *   score_t = q[i, h, :] . k[t, h / (H / G), :] * scale - slopes[h] * (row_pos[i] - t),  t <= row_pos[i]
+ *   out[i, h, :] = sum_t softmax(score)_t v[t, h / (H / G), :]
+ * slopes (fp32 [H], NULL: no bias).  span is an upper bound of the tokens a row sees; the rows' own tokens are in the cache
+ * already.  bf16 with dim and vdim multiples of 8 up to 128 runs on the tensor cores (the window of a row is cut into shares whose
+ * partial results go to a workspace of b2kv_gqa_decode_workspace_bytes bytes), everything else on CUDA cores (dim and vdim
+ * up to 512).  path: 0 = choose, 1 = CUDA cores, 2 = tensor cores.
+ */
+size_t b2kv_gqa_decode_workspace_bytes(int rows, int H, int G, int vdim, int span, int dtype);
+int b2kv_gqa_decode(const void* q, int64_t ld_q, const void* k_cache, const void* v_cache, void* out, int64_t ld_out,
+                    const float* slopes, const int32_t* row_slot, const int32_t* row_pos, int n_slots, int T_max, int rows, int H,
+                    int G, int dim, int vdim, int span, float scale, int dtype, int path, void* workspace,
+                    size_t workspace_bytes, int32_t* dev_status, void* stream);
+
+/*
+ * The same for prompt portions (bf16, tensor cores): segments as for b2kv_latent_prefill, with kv_row0 = cache_row0 = the
+ * first cache row of the segment's sequence.  b2kv_gqa_prefill_supported says whether the sizes have this form (dim and vdim
+ * multiples of 8 up to 128).
+ */
+int b2kv_gqa_prefill_supported(int dim, int vdim, int dtype);
+int b2kv_gqa_prefill(const void* q, int64_t ld_q, const void* k_cache, const void* v_cache, int64_t cache_rows, void* out,
+                     int64_t ld_out, const float* slopes, const b2kv_prompt_segment* segments, int n_segments, int n_blocks,
+                     int rows, int H, int G, int dim, int vdim, float scale, int dtype, int32_t* dev_status, void* stream);
+
+/*
+ * Gated linear attention: a recurrence whose state S [dim, vdim] (fp32, per sequence and head) forgets per key channel.
+ * For the rows of a segment in turn, per head, with q = y[:, q_col + h * dim ...] * q_scale, k and v likewise:
+ *   alpha = sigmoid(z)^(1 / tau)                     z fp32 [rows, H * dim]
+ *   S <- diag(alpha) S + k v^T,  o = S^T q
+ *   out[row, h, :] = o / sqrt(mean(o^2) + eps) * norm * silu(y[row, g_col + h * vdim ...])
+ * state [n_slots, H, dim, vdim] is read at the start of a segment (taken as zero where its first row's row_pos is 0) and
+ * written at its end.  segments (device): rows row0 .. row0 + n - 1 belong to sequence `slot`, in order; NULL: row i is a
+ * segment of its own, of sequence i.  max_n bounds the segments' lengths.  Everything is computed in 32-bit; path 2 (segments
+ * of a prompt; bf16, dim a multiple of 8 up to 128, vdim a multiple of 8 up to 256) takes sixteen tokens at a time through the tensor
+ * cores with operands split into two bf16 halves and the state in fp32 registers, path 1 takes token after token on CUDA
+ * cores for any sizes and both types; 0 = choose.
+ */
+typedef struct b2kv_row_segment {
+    int32_t row0, n, slot;
+} b2kv_row_segment;
+typedef struct b2kv_gla_args {
+    const void* y;
+    const float* z;
+    const float* norm;
+    float* state;
+    void* out;
+    const b2kv_row_segment* segments;
+    const int32_t* row_pos;
+    int64_t ld_y, ld_z, ld_out;
+    int32_t q_col, k_col, v_col, g_col;
+    int32_t H, dim, vdim, n_segments, max_n, rows, n_slots, dtype, path;
+    float q_scale, tau, eps;
+} b2kv_gla_args;
+int b2kv_gla(const b2kv_gla_args* args, int32_t* dev_status, void* stream);
 
 /*
  * Mixture of experts.  b2kv_route: per row of logits [rows, ld] (fp32, `experts` of them used): softmax over all experts,

@@ -37,7 +37,7 @@ _sz = ctypes.c_size_t
 
 _f = ctypes.c_float
 
-SEG_STORE, SEG_F32, SEG_GLU_SILU, SEG_GLU_CLAMP = 0, 1, 2, 3
+SEG_STORE, SEG_F32, SEG_GLU_SILU, SEG_GLU_CLAMP, SEG_RELU2, SEG_SOFTCAP = 0, 1, 2, 3, 4, 5
 MAX_SEGMENTS = 3
 
 
@@ -50,11 +50,22 @@ class Segment(ctypes.Structure):
 class LinearArgs(ctypes.Structure):
     """``b2kv_linear_args``."""
 
-    _fields_ = [("x", _vp), ("w", _vp), ("residual", _vp), ("group_rows", _vp), ("ld_x", _i64), ("group_x", _i64),
+    _fields_ = [("x", _vp), ("w", _vp), ("residual", _vp), ("bias", _vp), ("group_rows", _vp), ("ld_x", _i64), ("group_x", _i64),
                 ("ld_w", _i64), ("group_w", _i64), ("ld_residual", _i64), ("seg", Segment * MAX_SEGMENTS),
                 ("rows", ctypes.c_int32), ("K", ctypes.c_int32), ("N", ctypes.c_int32), ("groups", ctypes.c_int32),
                 ("max_group_rows", ctypes.c_int32), ("n_seg", ctypes.c_int32), ("dtype", ctypes.c_int32),
                 ("path", ctypes.c_int32), ("limit", _f)]
+
+
+class GlaArgs(ctypes.Structure):
+    """``b2kv_gla_args``."""
+
+    _fields_ = [("y", _vp), ("z", _vp), ("norm", _vp), ("state", _vp), ("out", _vp), ("segments", _vp), ("row_pos", _vp),
+                ("ld_y", _i64), ("ld_z", _i64), ("ld_out", _i64), ("q_col", ctypes.c_int32), ("k_col", ctypes.c_int32),
+                ("v_col", ctypes.c_int32), ("g_col", ctypes.c_int32), ("H", ctypes.c_int32), ("dim", ctypes.c_int32),
+                ("vdim", ctypes.c_int32), ("n_segments", ctypes.c_int32), ("max_n", ctypes.c_int32), ("rows", ctypes.c_int32),
+                ("n_slots", ctypes.c_int32), ("dtype", ctypes.c_int32), ("path", ctypes.c_int32), ("q_scale", _f), ("tau", _f),
+                ("eps", _f)]
 
 
 # name -> (restype, argtypes); kept in the order of include/b2kv.h
@@ -96,7 +107,8 @@ SIGNATURES = {
     "b2kv_qkv_append": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i64, _i64, _i64, _i, _vp, _vp]),
     "b2kv_matmul_rows": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp]),
     "b2kv_matmul": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp]),
-    "b2kv_embed_rows": (_i, [_vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp]),
+    "b2kv_embed_rows": (_i, [_vp, _vp, _vp, _vp, _f, _i, _i, _i, _i, _vp, _vp]),
+    "b2kv_layernorm_rows": (_i, [_vp, _i64, _vp, _vp, _vp, _vp, _i64, _vp, _i64, _i, _i, _f, _i, _vp]),
     "b2kv_rmsnorm": (_i, [_vp, _i64, _vp, _vp, _f, _vp, _i64, _i, _i, _f, _i, _vp]),
     "b2kv_linear": (_i, [ctypes.POINTER(LinearArgs), _vp, _vp]),
     "b2kv_latent_append": (_i, [_vp, _i64, _i, _i, _i, _i, _vp, _i, _i, _vp, _f, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp]),
@@ -106,6 +118,13 @@ SIGNATURES = {
     "b2kv_latent_prefill_supported": (_i, [_i, _i, _i, _i, _i]),
     "b2kv_latent_prefill": (_i, [_vp, _i64, _vp, _vp, _i64, _vp, _i64, _vp, _i64, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i,
                                  _vp, _vp]),
+    "b2kv_gqa_append": (_i, [_vp, _i64, _i, _i, _i, _i, _vp, _vp, _f, _f, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp]),
+    "b2kv_gqa_decode_workspace_bytes": (_sz, [_i, _i, _i, _i, _i, _i]),
+    "b2kv_gqa_decode": (_i, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _sz,
+                             _vp, _vp]),
+    "b2kv_gqa_prefill_supported": (_i, [_i, _i, _i]),
+    "b2kv_gqa_prefill": (_i, [_vp, _i64, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp]),
+    "b2kv_gla": (_i, [ctypes.POINTER(GlaArgs), _vp, _vp]),
     "b2kv_route": (_i, [_vp, _i64, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp]),
     "b2kv_moe_plan": (_i, [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _i64, _vp, _i64, _i, _i, _vp]),
     "b2kv_moe_combine": (_i, [_vp, _i64, _vp, _i64, _vp, _vp, _i, _i, _i, _i, _vp]),

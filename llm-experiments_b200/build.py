@@ -22,7 +22,7 @@ INCLUDE = PKG.parent / "include"
 OUT = PKG / "libb2kv.so"
 SERVE_OUT = PKG / "libb2kv_serve.so"
 OBJ_DIR = PKG / "build"
-SERVE_SOURCES = ("api", "append", "gemm", "latent", "latent_decode_tc", "latent_prefill", "linear", "linear_rows", "moe", "rows",
+SERVE_SOURCES = ("api", "append", "gemm", "gla", "gla_chunked", "gqa", "gqa_decode_tc", "latent", "latent_decode_tc", "latent_prefill", "linear", "linear_rows", "moe", "rows",
                  "step_tail")
 
 NVCC_FLAGS = [

@@ -78,7 +78,7 @@ const char* b2kv_strerror(int status) {
 
 const char* b2kv_last_cuda_error(void) { return b2kv::g_last_error; }
 
-int b2kv_version(void) { return 2; }
+int b2kv_version(void) { return 3; }
 
 int b2kv_tune(const char* name, int value) {
     if (name == nullptr) return B2KV_ERR_BAD_ARG;

@@ -438,9 +438,27 @@ __device__ __forceinline__ void epilogue_rows(const SegParams& p, uint32_t t_add
         tmem_wait_ld();
         if (!live) continue;
         const int64_t row = grow;
-        if (sg.kind == B2KV_SEG_F32) {
+        if (p.a.bias != nullptr) {
+#pragma unroll
+            for (int v = 0; v < 8; ++v) {
+                if (col0 + v * 4 >= p.N) break;  // (columns come in fours)
+                const float4 b = __ldg(reinterpret_cast<const float4*>(p.a.bias + col0 + v * 4));
+                acc[v * 4 + 0] = __float_as_uint(__uint_as_float(acc[v * 4 + 0]) + b.x);
+                acc[v * 4 + 1] = __float_as_uint(__uint_as_float(acc[v * 4 + 1]) + b.y);
+                acc[v * 4 + 2] = __float_as_uint(__uint_as_float(acc[v * 4 + 2]) + b.z);
+                acc[v * 4 + 3] = __float_as_uint(__uint_as_float(acc[v * 4 + 3]) + b.w);
+            }
+        }
+        if (sg.kind == B2KV_SEG_RELU2) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) acc[i] = __float_as_uint(lin::single(B2KV_SEG_RELU2, __uint_as_float(acc[i]), 0.f));
+        } else if (sg.kind == B2KV_SEG_SOFTCAP) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) acc[i] = __float_as_uint(lin::single(B2KV_SEG_SOFTCAP, __uint_as_float(acc[i]), p.a.limit));
+        }
+        if (lin::is_f32(sg.kind)) {
             float* out = static_cast<float*>(sg.out) + row * sg.ld + local;
-            const float* res = p.a.residual ? p.a.residual + row * p.a.ld_residual + local : nullptr;
+            const float* res = p.a.residual && sg.kind == B2KV_SEG_F32 ? p.a.residual + row * p.a.ld_residual + local : nullptr;
             float4 add[8];
 #pragma unroll
             for (int v = 0; v < 8; ++v)
@@ -454,7 +472,7 @@ __device__ __forceinline__ void epilogue_rows(const SegParams& p, uint32_t t_add
                 o.z = __uint_as_float(acc[v * 4 + 2]) + add[v].z, o.w = __uint_as_float(acc[v * 4 + 3]) + add[v].w;
                 *reinterpret_cast<float4*>(out + v * 4) = o;
             }
-        } else if (sg.kind == B2KV_SEG_STORE) {
+        } else if (!lin::is_pair(sg.kind)) {
             __nv_bfloat16* out = static_cast<__nv_bfloat16*>(sg.out) + row * sg.ld + local;
 #pragma unroll
             for (int v = 0; v < 4; ++v) {
@@ -742,11 +760,12 @@ int b2kv::linear_tiled_tc(const b2kv_linear_args& a, int32_t* dev_status, void* 
     int first = 0;
     for (int s = 0; s < a.n_seg; ++s) {  // 16-byte accesses in the epilogue; 32 columns lie in one segment
         const b2kv_segment& sg = a.seg[s];
-        const bool f32 = sg.kind == B2KV_SEG_F32, glu = sg.kind >= B2KV_SEG_GLU_SILU;
+        const bool f32 = lin::is_f32(sg.kind), glu = lin::is_pair(sg.kind);
         if (first % 32 != 0 || (sg.end - first) % (glu ? 16 : (f32 ? 4 : 8)) != 0) return B2KV_ERR_UNSUPPORTED;
         if (!aligned16(sg.out) || sg.ld % (f32 ? 4 : 8) != 0) return B2KV_ERR_UNSUPPORTED;
         first = sg.end;
     }
+    if (a.bias && !aligned16(a.bias)) return B2KV_ERR_UNSUPPORTED;
     if (a.residual && (!aligned16(a.residual) || a.ld_residual % 4 != 0)) return B2KV_ERR_UNSUPPORTED;
     gemm::SegParams p{a, a.rows, a.N, a.K, 0, 0, dev_status};
     // with groups the number of tiles is only known on the device: every group may end in a partly filled tile

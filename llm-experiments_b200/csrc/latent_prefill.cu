@@ -1,4 +1,5 @@
-// Attention of prompt portions over keys and values expanded from cached latent rows, on the Blackwell tensor cores (bf16).
+// Attention of prompt portions on the Blackwell tensor cores (bf16): over keys and values expanded from cached latent rows, and over
+// cached keys and values of grouped heads.
 //
 // The scheme is that of prefill_tc.cu: one CTA per head and 256 query rows (two 128-row tiles A and B that share every 128-key
 // tile), warp 8 copies with TMA, warp 9 issues tcgen05.mma (S = Q K^T from shared memory, O += P V with P read from tensor
@@ -18,10 +19,14 @@
 //     chunk (a ring of two) and a pair, V tiles a pair, the pairs form one ring of three that K(0) V(0) K(1) V(1) ... pass
 //     through.  K(j + 1) and V(j + 1) are then on their way while K(j) and V(j) are in use.
 //
+// Grouped heads (no rotated part) read the caches in place: key row t of a segment is a cache row, head h takes the columns of
+// key / value head h / (H / G).  A distance bias, slope_h * (query position - key position), is taken off the scores in fp32.
+//
 // TMEM columns: S_A 0-127, S_B 128-255, O_A 256-383, O_B 384-511.  Every wait is bounded.
 #include <math.h>
 
 #include <algorithm>
+#include <type_traits>
 
 #include "tc_ptx.cuh"
 #include "tma_map.cuh"
@@ -43,16 +48,18 @@ struct Params {
     __nv_bfloat16* out;  // row i of the step at out + i * ld_out, head h at column h * vdim
     const b2kv_prompt_segment* seg;
     int32_t* dev_status;
+    const float* slopes;  // fp32 [H], with kBias
     int64_t ld_out;
     int n_seg, n_blocks, H, group, dim, rot, vdim, window;
-    float prescale;
-    int rows, kv_rows, cache_rows;  // scale * log2(e)
+    float prescale;  // scale * log2(e)
+    int rows, kv_rows, cache_rows;
+    int per_kv;  // query heads per key / value head
 };
 
-// kNope + 1 chunks per key (the last one is the rotated part), kV chunks per value.
-template <int kNope, int kV>
+// kNope chunks per key, with kRot one more for the rotated part; kV chunks per value.
+template <int kNope, bool kRot, int kV>
 struct Storage {
-    static constexpr int kK = kNope + 1;
+    static constexpr int kK = kNope + (kRot ? 1 : 0);
     static constexpr bool kSharedRing = kK == 3 && kV == 2;
     static constexpr int kChunks = kSharedRing ? 8 : 2 * (kK + kV);
     alignas(1024) uint8_t q[2][kK][kChunkBytes];
@@ -74,13 +81,13 @@ struct Storage {
     }
 };
 
-template <int kNope, int kV>
+template <int kNope, bool kRot, int kV, bool kBias>
 __global__ void __launch_bounds__(kThreads, 1)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
                       const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
                       const __grid_constant__ CUtensorMap tm_v, const Params p) {
     extern __shared__ uint8_t smem_raw[];
-    using Smem = Storage<kNope, kV>;
+    using Smem = Storage<kNope, kRot, kV>;
     constexpr int kK = Smem::kK;
     Smem& sm = *reinterpret_cast<Smem*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -92,6 +99,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
     const int within = static_cast<int>(blockIdx.x) - gi * per_group;
     const int block = p.n_blocks - 1 - within / heads_here;
     const int h = gi * p.group + within % heads_here;
+    const int h_kv = kRot ? h : h / p.per_kv;
     int si = 0;
     while (si + 1 < p.n_seg && p.seg[si + 1].first_block <= block) ++si;
     const b2kv_prompt_segment sg = p.seg[si];
@@ -143,7 +151,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
                 const int row = sg.row0 + q0 + x * kTileM;
 #pragma unroll
                 for (int c = 0; c < kNope; ++c) tma_load_3d(sm.q[x][c], &tm_qn, &sm.q_full, c * 64, h, row);
-                tma_load_3d(sm.q[x][kNope], &tm_qr, &sm.q_full, 0, h, row);
+                if (kRot) tma_load_3d(sm.q[x][kK - 1], &tm_qr, &sm.q_full, 0, h, row);
             }
             bool ok = true;
             for (int j = 0; j < n_tiles; ++j) {
@@ -156,8 +164,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
                 mbar_arrive_expect_tx(&sm.k_full[st], kK * kChunkBytes);
 #pragma unroll
                 for (int c = 0; c < kNope; ++c)
-                    tma_load_3d(sm.kv[Smem::k_chunk(j, c)], &tm_kn, &sm.k_full[st], c * 64, h, sg.kv_row0 + key);
-                tma_load_3d(sm.kv[Smem::k_chunk(j, kNope)], &tm_kr, &sm.k_full[st], 0, 0, sg.cache_row0 + key);
+                    tma_load_3d(sm.kv[Smem::k_chunk(j, c)], &tm_kn, &sm.k_full[st], c * 64, h_kv, sg.kv_row0 + key);
+                if (kRot) tma_load_3d(sm.kv[Smem::k_chunk(j, kNope)], &tm_kr, &sm.k_full[st], 0, 0, sg.cache_row0 + key);
                 ok = mbar_wait(&sm.v_empty[st], par);
                 // K(j - 1) leaves its pair to V(j)
                 if (Smem::kSharedRing && ok && j > 0) ok = mbar_wait(&sm.k_empty[st ^ 1], ((j - 1) >> 1) & 1);
@@ -165,7 +173,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
                 mbar_arrive_expect_tx(&sm.v_full[st], kV * kChunkBytes);
 #pragma unroll
                 for (int c = 0; c < kV; ++c)
-                    tma_load_3d(sm.kv[Smem::v_chunk(j) + c], &tm_v, &sm.v_full[st], c * 64, h, sg.kv_row0 + key);
+                    tma_load_3d(sm.kv[Smem::v_chunk(j) + c], &tm_v, &sm.v_full[st], c * 64, h_kv, sg.kv_row0 + key);
             }
             if (!ok) sm.abort_flag = 1;
         }
@@ -191,7 +199,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
 #pragma unroll
                     for (int kk = 0; kk < 4; ++kk)
                         mma_ss(s_tmem, a + static_cast<uint64_t>(c * kChunk16 + 2 * kk),
-                               c == kNope ? b_last + static_cast<uint64_t>(2 * kk) : b + static_cast<uint64_t>(c * kChunk16 + 2 * kk),
+                               kRot && c == kNope ? b_last + static_cast<uint64_t>(2 * kk) : b + static_cast<uint64_t>(c * kChunk16 + 2 * kk),
                                idesc_qk, (c | kk) ? 1u : 0u);
                 }
                 mma_commit(&sm.s_full[x]);
@@ -257,6 +265,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
         const uint32_t s_tmem = tmem + lane_base + kColS + x * 128;
         const uint32_t o_tmem = tmem + lane_base + kColO + x * 128;
         const float c = p.prescale;
+        const float slope = kBias ? p.slopes[h] * 1.4426950408889634f : 0.f;
         const int own = sg.own + q0 + x * kTileM;  // key row of the tile's first query
         float m_used = -INFINITY, m_run = -INFINITY, l = 0.f;
         bool ok = true;
@@ -271,6 +280,19 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
             // columns this row sees: [lo, hi]; a tile that every row of the row tile sees whole needs no mask
             const int hi = own + row - key0;
             const int lo = p.window > 0 ? hi - p.window + 1 : -1;
+            const float2 c2 = make_float2(c, c);
+            if (kBias) {
+                // element e is hi - e tokens behind the query
+                const float base = -slope * static_cast<float>(hi);
+                const float2 slope2 = make_float2(slope, slope), base2 = make_float2(base, base);
+#pragma unroll
+                for (int e = 0; e < 128; e += 2) {
+                    const float2 b = __ffma2_rn(make_float2(static_cast<float>(e), static_cast<float>(e + 1)), slope2, base2);
+                    const float2 z = __ffma2_rn(make_float2(__uint_as_float(r[e]), __uint_as_float(r[e + 1])), c2, b);
+                    r[e] = __float_as_uint(z.x);
+                    r[e + 1] = __float_as_uint(z.y);
+                }
+            }
             if (key0 + kBlockN - 1 > own || (p.window > 0 && own + kTileM - 1 - p.window + 1 > key0)) {
 #pragma unroll
                 for (int e = 0; e < 128; ++e)
@@ -283,7 +305,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
             for (int e = 8; e < 128; ++e) mxs[e & 7] = fmaxf(mxs[e & 7], __uint_as_float(r[e]));
             const float mx = fmaxf(fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3])),
                                    fmaxf(fmaxf(mxs[4], mxs[5]), fmaxf(mxs[6], mxs[7])));
-            m_run = fmaxf(m_run, mx * c);
+            m_run = fmaxf(m_run, kBias ? mx : mx * c);
             float factor = 1.f;
             bool need = false;
             if (i == 0) {
@@ -298,13 +320,14 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
             float sums[8];
 #pragma unroll
             for (int a = 0; a < 8; ++a) sums[a] = 0.f;
-            const float2 c2 = make_float2(c, c), neg_m2 = make_float2(neg_m, neg_m);
+            const float2 neg_m2 = make_float2(neg_m, neg_m);
 #pragma unroll
             for (int cc = 0; cc < 4; ++cc) {
                 uint32_t pk[16];
 #pragma unroll
                 for (int e = 0; e < 16; ++e) {
-                    const float2 z = __ffma2_rn(make_float2(__uint_as_float(r[cc * 32 + 2 * e]), __uint_as_float(r[cc * 32 + 2 * e + 1])), c2, neg_m2);
+                    const float2 s2 = make_float2(__uint_as_float(r[cc * 32 + 2 * e]), __uint_as_float(r[cc * 32 + 2 * e + 1]));
+                    const float2 z = kBias ? __fadd2_rn(s2, neg_m2) : __ffma2_rn(s2, c2, neg_m2);
                     const float p0 = ex2(z.x), p1 = ex2(z.y);
                     sums[(2 * e) & 7] += p0;
                     sums[(2 * e + 1) & 7] += p1;
@@ -388,11 +411,11 @@ static bool make_map(CUtensorMap* map, const void* base, int width, int heads, i
               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int kNope, int kV>
+template <int kNope, bool kRot, int kV, bool kBias>
 static int launch(const CUtensorMap (&m)[5], const Params& p, long long ctas, void* stream) {
-    constexpr size_t smem = sizeof(Storage<kNope, kV>) + 1024;
+    constexpr size_t smem = sizeof(Storage<kNope, kRot, kV>) + 1024;
     static_assert(smem <= 227 * 1024, "the tiles must fit one SM's shared memory");
-    auto kernel = latent_prefill_kernel<kNope, kV>;
+    auto kernel = latent_prefill_kernel<kNope, kRot, kV, kBias>;
     static bool configured[64] = {false};
     int dev = 0;
     B2KV_CUDA_TRY(cudaGetDevice(&dev));
@@ -436,13 +459,50 @@ extern "C" int b2kv_latent_prefill(const void* q, int64_t ld_q, const void* keys
         !make_map(&m[2], keys, dim, H, kv_rows, dim, ld_kv) || !make_map(&m[3], key_cache, rot, 1, cache_rows, rot, rot) ||
         !make_map(&m[4], values, vdim, H, kv_rows, vdim, ld_kv))
         return B2KV_ERR_UNSUPPORTED;
-    Params p{static_cast<__nv_bfloat16*>(out), segments, dev_status, ld_out, n_segments, n_blocks, H, 0, dim, rot, vdim, window,
-             scale * 1.4426950408889634f, rows, kv_rows, static_cast<int>(cache_rows)};
+    Params p{static_cast<__nv_bfloat16*>(out), segments, dev_status, nullptr, ld_out, n_segments, n_blocks, H, 0, dim, rot, vdim,
+             window, scale * 1.4426950408889634f, rows, kv_rows, static_cast<int>(cache_rows), 1};
     // heads whose keys and values together take about 32 MB, a quarter of L2, run next to each other
     const long long head_bytes = 2LL * kv_rows * (dim + vdim);
     p.group = static_cast<int>(std::min<long long>(H, std::max<long long>(1, (32LL << 20) / head_bytes)));
     const long long ctas = static_cast<long long>(n_blocks) * H;
     if (ctas > 0x7fffffffLL) return B2KV_ERR_UNSUPPORTED;
-    if (dim <= 64) return vdim <= 64 ? launch<1, 1>(m, p, ctas, stream) : launch<1, 2>(m, p, ctas, stream);
-    return vdim <= 64 ? launch<2, 1>(m, p, ctas, stream) : launch<2, 2>(m, p, ctas, stream);
+    if (dim <= 64) return vdim <= 64 ? launch<1, true, 1, false>(m, p, ctas, stream) : launch<1, true, 2, false>(m, p, ctas, stream);
+    return vdim <= 64 ? launch<2, true, 1, false>(m, p, ctas, stream) : launch<2, true, 2, false>(m, p, ctas, stream);
+}
+
+extern "C" int b2kv_gqa_prefill_supported(int dim, int vdim, int dtype) {
+    return dtype == B2KV_DTYPE_BF16 && dim > 0 && dim <= 128 && dim % 8 == 0 && vdim > 0 && vdim <= 128 && vdim % 8 == 0;
+}
+
+extern "C" int b2kv_gqa_prefill(const void* q, int64_t ld_q, const void* k_cache, const void* v_cache, int64_t cache_rows, void* out,
+                                int64_t ld_out, const float* slopes, const b2kv_prompt_segment* segments, int n_segments,
+                                int n_blocks, int rows, int H, int G, int dim, int vdim, float scale, int dtype,
+                                int32_t* dev_status, void* stream) {
+    using namespace latpre;
+    if (!q || !k_cache || !v_cache || !out || !segments || n_segments <= 0 || n_blocks <= 0 || rows <= 0 || cache_rows <= 0 ||
+        cache_rows > 0x7fffff00LL || H <= 0 || G <= 0 || H % G != 0)
+        return B2KV_ERR_BAD_ARG;
+    if (!b2kv_gqa_prefill_supported(dim, vdim, dtype) || !(scale > 0.f)) return B2KV_ERR_UNSUPPORTED;
+    if (ld_q < static_cast<int64_t>(H) * dim || ld_out < static_cast<int64_t>(H) * vdim) return B2KV_ERR_BAD_ARG;
+    if (!aligned16(q) || !aligned16(k_cache) || !aligned16(v_cache) || !aligned16(out) || ld_q % 8 || ld_out % 8) return B2KV_ERR_ALIGN;
+    CUtensorMap m[5];
+    if (!make_map(&m[0], q, dim, H, rows, dim, ld_q) ||
+        !make_map(&m[2], k_cache, dim, G, cache_rows, dim, static_cast<int64_t>(G) * dim) ||
+        !make_map(&m[4], v_cache, vdim, G, cache_rows, vdim, static_cast<int64_t>(G) * vdim))
+        return B2KV_ERR_UNSUPPORTED;
+    m[1] = m[0], m[3] = m[2];  // (no rotated parts: not used)
+    const int per_kv = H / G;
+    Params p{static_cast<__nv_bfloat16*>(out), segments, dev_status, slopes, ld_out, n_segments, n_blocks, H, 0, dim, 0, vdim,
+             0, scale * 1.4426950408889634f, rows, static_cast<int>(cache_rows), static_cast<int>(cache_rows), per_kv};
+    // heads whose keys and values of the step's own tokens take about 32 MB run next to each other
+    const long long head_bytes = 2LL * rows * (dim + vdim);
+    p.group = static_cast<int>(std::min<long long>(H, std::max<long long>(1, (32LL << 20) / head_bytes) * per_kv));
+    const long long ctas = static_cast<long long>(n_blocks) * H;
+    if (ctas > 0x7fffffffLL) return B2KV_ERR_UNSUPPORTED;
+    auto go = [&](auto bias) {
+        constexpr bool kBias = decltype(bias)::value;
+        if (dim <= 64) return vdim <= 64 ? launch<1, false, 1, kBias>(m, p, ctas, stream) : launch<1, false, 2, kBias>(m, p, ctas, stream);
+        return vdim <= 64 ? launch<2, false, 1, kBias>(m, p, ctas, stream) : launch<2, false, 2, kBias>(m, p, ctas, stream);
+    };
+    return slopes != nullptr ? go(std::true_type{}) : go(std::false_type{});
 }

@@ -72,7 +72,11 @@ __global__ void __launch_bounds__(kThreads) linear_simt_kernel(const b2kv_linear
             const b2kv_segment& sg = a.seg[s];
             const int local = c - segment_first(a, s);
             const int64_t base = out_row * sg.ld + static_cast<int64_t>(g) * (a.group_rows ? 0 : sg.group);
-            if (sg.kind >= B2KV_SEG_GLU_SILU) {
+            if (a.bias != nullptr) {
+                acc[i][j] += a.bias[c];
+                if (c + 1 < a.N) acc[i][j + 1] += a.bias[c + 1];
+            }
+            if (is_pair(sg.kind)) {
                 static_cast<T*>(sg.out)[base + local / 2] =
                     Elt<T>::from_float(glu_value<T>(sg.kind, acc[i][j], acc[i][j + 1], a.limit));
                 continue;
@@ -80,9 +84,9 @@ __global__ void __launch_bounds__(kThreads) linear_simt_kernel(const b2kv_linear
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 if (c + e >= a.N) break;
-                float v = acc[i][j + e];
-                if (sg.kind == B2KV_SEG_F32) {
-                    if (a.residual != nullptr) v += a.residual[out_row * a.ld_residual + local + e];
+                float v = single(sg.kind, acc[i][j + e], a.limit);
+                if (is_f32(sg.kind)) {
+                    if (a.residual != nullptr && sg.kind == B2KV_SEG_F32) v += a.residual[out_row * a.ld_residual + local + e];
                     static_cast<float*>(sg.out)[base + local + e] = v;
                 } else {
                     static_cast<T*>(sg.out)[base + local + e] = Elt<T>::from_float(v);
@@ -115,7 +119,7 @@ static int rows_in_slices(const b2kv_linear_args& all, int32_t* dev_status, void
         a.x = static_cast<const char*>(all.x) + r0 * all.ld_x * es;
         if (all.residual) a.residual = all.residual + r0 * all.ld_residual;
         for (int s = 0; s < a.n_seg; ++s)
-            a.seg[s].out = static_cast<char*>(all.seg[s].out) + r0 * all.seg[s].ld * (all.seg[s].kind == B2KV_SEG_F32 ? 4 : es);
+            a.seg[s].out = static_cast<char*>(all.seg[s].out) + r0 * all.seg[s].ld * (is_f32(all.seg[s].kind) ? 4 : es);
         const int rc = linear_rows_tc(a, dev_status, stream);
         if (rc != B2KV_OK) return rc;
     }
@@ -133,13 +137,14 @@ extern "C" int b2kv_linear(const b2kv_linear_args* args, int32_t* dev_status, vo
     if (elt_bytes(a.dtype) == 0) return B2KV_ERR_UNSUPPORTED;
     if (!a.x || !a.w || a.rows <= 0 || a.K <= 0 || a.N <= 0 || a.groups <= 0 || a.path < 0 || a.path > 3) return B2KV_ERR_BAD_ARG;
     if (a.n_seg < 1 || a.n_seg > B2KV_MAX_SEGMENTS || a.seg[a.n_seg - 1].end != a.N) return B2KV_ERR_BAD_ARG;
+    if (a.bias && a.groups > 1) return B2KV_ERR_BAD_ARG;
     if (a.group_rows && (a.max_group_rows <= 0 || a.max_group_rows > a.rows)) return B2KV_ERR_BAD_ARG;
     int first = 0;
     for (int s = 0; s < a.n_seg; ++s) {
         const b2kv_segment& sg = a.seg[s];
-        if (!sg.out || sg.end <= first || sg.kind < B2KV_SEG_STORE || sg.kind > B2KV_SEG_GLU_CLAMP) return B2KV_ERR_BAD_ARG;
+        if (!sg.out || (sg.kind == B2KV_SEG_SOFTCAP && !(a.limit > 0.f)) || sg.end <= first || sg.kind < B2KV_SEG_STORE || sg.kind > B2KV_SEG_SOFTCAP) return B2KV_ERR_BAD_ARG;
         // pairs of columns never straddle a boundary (the last segment may end on an odd column if it has no pairs)
-        if ((sg.end & 1) && (s + 1 < a.n_seg || sg.kind >= B2KV_SEG_GLU_SILU)) return B2KV_ERR_BAD_ARG;
+        if ((sg.end & 1) && (s + 1 < a.n_seg || lin::is_pair(sg.kind))) return B2KV_ERR_BAD_ARG;
         first = sg.end;
     }
     if (a.path == 2) return linear_rows_tc(a, dev_status, stream);

@@ -14,6 +14,19 @@ __device__ __forceinline__ float glu(int kind, float g, float u, float limit) {
     return g / (1.0f + __expf(-1.702f * g)) * (u + 1.0f);
 }
 
+// Kinds whose columns are (gate, up) pairs; kinds whose output is fp32.
+__host__ __device__ constexpr bool is_pair(int kind) { return kind == B2KV_SEG_GLU_SILU || kind == B2KV_SEG_GLU_CLAMP; }
+__host__ __device__ constexpr bool is_f32(int kind) { return kind == B2KV_SEG_F32 || kind == B2KV_SEG_SOFTCAP; }
+
+// What happens to a single column before it is stored.
+__device__ __forceinline__ float single(int kind, float v, float limit) {
+    if (kind == B2KV_SEG_RELU2) {
+        v = fmaxf(v, 0.f);
+        return v * v;
+    }
+    return kind == B2KV_SEG_SOFTCAP ? limit * tanhf(v / limit) : v;
+}
+
 // Index of the segment that holds column c (segments are in column order).
 __device__ __forceinline__ int segment_of(const b2kv_linear_args& a, int c) {
     int s = 0;

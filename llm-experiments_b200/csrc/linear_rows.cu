@@ -72,13 +72,16 @@ struct Place {
     const float* residual;
     int64_t ld, ld_residual, col;  // col: element inside the output row
     int kind;
+    float bias;
     bool live;
 };
 
 // Stores kN values of this thread's feature, for rows row[0 .. kN - 1] (-1: none).
 template <int kN>
-__device__ __forceinline__ void emit(const Place& pl, const float (&v)[kN], const int64_t (&row)[kN], float limit) {
-    if (pl.kind >= B2KV_SEG_GLU_SILU) {
+__device__ __forceinline__ void emit(const Place& pl, float (&v)[kN], const int64_t (&row)[kN], float limit) {
+#pragma unroll
+    for (int j = 0; j < kN; ++j) v[j] += pl.bias;
+    if (lin::is_pair(pl.kind)) {
         // (kind is the same for the whole warp: segments start on multiples of 32 columns)
         const bool odd = threadIdx.x & 1;
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(pl.out) + pl.col;
@@ -93,7 +96,11 @@ __device__ __forceinline__ void emit(const Place& pl, const float (&v)[kN], cons
         return;
     }
     if (!pl.live) return;
-    if (pl.kind == B2KV_SEG_F32) {
+    if (pl.kind >= B2KV_SEG_RELU2) {
+#pragma unroll
+        for (int j = 0; j < kN; ++j) v[j] = lin::single(pl.kind, v[j], limit);
+    }
+    if (lin::is_f32(pl.kind)) {
         float* out = static_cast<float*>(pl.out) + pl.col;
         float add[kN];
 #pragma unroll
@@ -271,9 +278,10 @@ linear_rows_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
         pl.out = sg.out;
         pl.ld = sg.ld;
         pl.ld_residual = p.a.ld_residual;
-        pl.col = (sg.kind >= B2KV_SEG_GLU_SILU ? local / 2 : local) + (by_rows ? 0 : static_cast<int64_t>(g) * sg.group);
+        pl.col = (lin::is_pair(sg.kind) ? local / 2 : local) + (by_rows ? 0 : static_cast<int64_t>(g) * sg.group);
         pl.residual = sg.kind == B2KV_SEG_F32 ? p.a.residual : nullptr;
         pl.live = c < p.a.N;
+        pl.bias = pl.live && p.a.bias != nullptr ? p.a.bias[c] : 0.f;
         if (p.splits > 1) {
             bool all = true;
             for (int sp = 0; sp < p.splits; ++sp) all = all && *reinterpret_cast<volatile int*>(&sm.got[sp]) == 1;

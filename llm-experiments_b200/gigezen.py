@@ -15,32 +15,30 @@ The concatenations are free: the two sublayers of a layer read the same rows and
 matrices stand side by side and their last ones on top of each other, and a layer is two weight-streaming launches beside its
 attention.  A layer may read another layer's cached latents (``kv_from``) with matrices of its own.
 
-A step runs any mix of sequences and portions: rows of (sequence, position), short entries first.  Every layer that owns
-latents has a ``KVCache`` of one layer; all share one tensor of lengths on the device.
+Steps, places and lengths are those of ``serving``.  Every layer that owns latents has a ``KVCache`` of one layer; all share one
+tensor of lengths on the device.  Short entries are attended row by row in the latent space; prompt portions expand the visible
+latents into keys and values first, which pays once several rows share them.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
-from typing import Dict, List, Optional, Sequence, Tuple
+from dataclasses import dataclass
+from typing import Dict, List, Optional
 
-import numpy as np
 import torch
 
 from . import latent, moe
-from ._native import lib as _lib
-from ._native import check as _check
-from .batch import batch_begin, batch_commit, batch_op_begin
 from .kv_cache import kv_cache_create
 from .latent import LatentShape, PromptPlan, RowPlaces
 from .moe import ExpertWeights, MoeScratch, RouterShape
 from .projection import SEG_F32, SEG_GLU_CLAMP, SEG_STORE, OutputSegment, linear
 from .registry import register_model
-from .step_tail import argmax, embedding_rows, rms_norm
+from .serving import SequenceState, ServedModel, Step, decode_step, forward, state_release, state_reset, state_set_lengths  # noqa: F401
+from .serving import buffer1 as _b1
+from .serving import buffer2 as _b2
+from .serving import pad_to as _pad
+from .serving import sub as _sub
+from .step_tail import embedding_rows, rms_norm
 from .types import GPUBuffer1D, GPUBuffer2D, GPUContext, KVCache, KVCacheConfig
-
-# Entries of at most this many tokens are attended row by row in the latent space; longer ones expand the visible latents
-# into keys and values first, which pays once several rows share them.
-SHORT_ENTRY = 16
 
 
 # ---------------------------------------------------------------------------------------------------------------
@@ -96,18 +94,6 @@ class GigezenConfig:
 # ---------------------------------------------------------------------------------------------------------------
 # weights
 # ---------------------------------------------------------------------------------------------------------------
-
-def _pad(n: int, to: int) -> int:
-    return (n + to - 1) // to * to
-
-
-def _b2(t: torch.Tensor) -> GPUBuffer2D:
-    return GPUBuffer2D(buffer=t, shape=tuple(t.shape), size=t.numel())
-
-
-def _b1(t: torch.Tensor) -> GPUBuffer1D:
-    return GPUBuffer1D(buffer=t, shape=tuple(t.shape), size=t.numel())
-
 
 @dataclass
 class LayerWeights:
@@ -234,47 +220,33 @@ def random_tensors(ctx: GPUContext, config: dict, seed: int = 0) -> Dict[str, to
 # ---------------------------------------------------------------------------------------------------------------
 
 @dataclass
-class GigezenState:
-    """Caches (one per layer that owns latents), lengths and scratch rows of ``batch_size`` sequences."""
+class GigezenState(SequenceState):
+    """One cache per layer that owns latents."""
 
-    cfg: GigezenConfig
-    weights: GigezenWeights
-    batch_size: int
-    max_seq_len: int
-    dtype: torch.dtype
-    owned: Dict[int, KVCache]
-    seq_lens: torch.Tensor           # int32 [batch_size] on the device, shared by all caches
-    lengths: List[int]               # the same on the host
-    scratch: Dict[str, torch.Tensor] = field(default_factory=dict)
-    prompt_form: bool = False        # every layer's sizes have a tensor-core form for prompt portions
-    logits: Optional[GPUBuffer2D] = None  # fp32 rows of the last step
-    layer_tap: Optional[list] = None      # debugging: receives a copy of the residual rows after every layer
-
-    @property
-    def caches(self) -> List[KVCache]:
-        return list(self.owned.values())
+    cfg: Optional[GigezenConfig] = None
+    weights: Optional[GigezenWeights] = None
 
     def cache_of(self, layer: int) -> KVCache:
         src = self.cfg.layers[layer].kv_from
         return self.owned[layer if src is None else src]
 
-    def rows(self, name: str, rows: int, cols: int, dtype: torch.dtype) -> GPUBuffer2D:
-        """The first ``rows`` rows of a scratch buffer that grows on demand.  It starts at zero: padding columns that nothing
-        writes are multiplied with zero weights and must be numbers."""
-        t = self.scratch.get(name)
-        if t is None or t.shape[0] < rows or t.shape[1] != cols:
-            t = torch.zeros((rows, cols), dtype=dtype, device=self.seq_lens.device)
-            self.scratch[name] = t
-        return GPUBuffer2D(buffer=t[:rows], shape=(rows, cols), size=rows * cols)
+    def prompt_plans(self, spans) -> Dict[int, PromptPlan]:
+        windows = sorted({lc.attention.window for lc in self.cfg.layers})
+        return {win: PromptPlan.build(spans, win, self.max_seq_len) for win in windows}
 
-    def advance_host(self, n: int = 1) -> None:
-        """Host-side part of advancing every sequence by ``n`` tokens."""
-        self.lengths = [v + n for v in self.lengths]
-        self._sync_upper_bound()
-
-    def _sync_upper_bound(self) -> None:
-        for c in self.owned.values():
-            c.current_len = max(self.lengths)
+    def run(self, ctx: GPUContext, step: Step) -> None:
+        cfg, w = self.cfg, self.weights
+        x = self.rows("x", step.rows, cfg.width, torch.float32)
+        embedding_rows(ctx, w.embedding, step.ids, x)
+        for i in range(len(cfg.layers)):
+            _layer(ctx, self, i, x, step)
+        if step.n_out == 0:
+            return
+        hl = self.rows("h_out", step.n_out, cfg.width, self.dtype)
+        rms_norm(ctx, x, w.final_norm, hl, cfg.eps, weight_offset=1.0, row_index=step.row_index)
+        out = self.rows("logits", step.n_out, cfg.vocab_size, torch.float32)
+        linear(ctx, hl, w.head, cfg.width, [OutputSegment(cfg.vocab_size, SEG_F32, out)])
+        self.logits = out
 
 
 def state_create(ctx: GPUContext, cfg: GigezenConfig, weights: GigezenWeights, batch_size: int, max_seq_len: int,
@@ -292,33 +264,9 @@ def state_create(ctx: GPUContext, cfg: GigezenConfig, weights: GigezenWeights, b
                         prompt_form=all(latent.prefill_supported(lc.attention, dtype) for lc in cfg.layers))
 
 
-def state_set_lengths(state: GigezenState, lens: Sequence[int]) -> None:
-    if len(lens) != state.batch_size or min(lens) < 0 or max(lens) > state.max_seq_len:
-        raise ValueError(f"lengths must be {state.batch_size} values in [0, {state.max_seq_len}]")
-    state.lengths = [int(v) for v in lens]
-    state.seq_lens.copy_(torch.tensor(state.lengths, dtype=torch.int32), non_blocking=False)
-    state._sync_upper_bound()
-
-
-def state_reset(state: GigezenState) -> None:
-    state_set_lengths(state, [0] * state.batch_size)
-
-
-def state_release(state: GigezenState, slot: int) -> None:
-    """Gives a finished sequence's place back: its cache rows are free for the next sequence."""
-    lens = list(state.lengths)
-    lens[slot] = 0
-    state_set_lengths(state, lens)
-
-
 # ---------------------------------------------------------------------------------------------------------------
 # the step
 # ---------------------------------------------------------------------------------------------------------------
-
-def _sub(b: GPUBuffer2D, r0: int, n: int, c0: int = 0, cols: Optional[int] = None) -> GPUBuffer2D:
-    cols = b.shape[1] - c0 if cols is None else cols
-    return GPUBuffer2D(buffer=b.buffer[r0:r0 + n, c0:c0 + cols], shape=(n, cols), size=n * cols)
-
 
 def _attend_rows(ctx, state: GigezenState, i: int, y: GPUBuffer2D, z: GPUBuffer2D, places: RowPlaces, span: int) -> None:
     """Attention of single rows in the latent space: per-head key matrix, latent attention, per-head value matrix."""
@@ -332,8 +280,7 @@ def _attend_rows(ctx, state: GigezenState, i: int, y: GPUBuffer2D, z: GPUBuffer2
            groups=a.heads, group_x=a.kv_rank, group_w=a.vdim)
 
 
-def _layer(ctx, state: GigezenState, i: int, x: GPUBuffer2D, places: RowPlaces, n_single: int, span: int,
-           plans: Dict[int, PromptPlan]) -> None:
+def _layer(ctx, state: GigezenState, i: int, x: GPUBuffer2D, step: Step) -> None:
     lc, w, T = state.cfg.layers[i], state.weights.layers[i], x.shape[0]
     a, cfg, dt = lc.attention, state.cfg, state.dtype
     cache = state.cache_of(i)
@@ -349,12 +296,12 @@ def _layer(ctx, state: GigezenState, i: int, x: GPUBuffer2D, places: RowPlaces, 
     if lc.dense_ff:
         segments.append(OutputSegment(w.y_cols + 2 * w.ff_cols, SEG_GLU_CLAMP, _sub(z, 0, T, w.a_cols)))
     linear(ctx, h, w.w_in, cfg.width, segments, limit=lc.limit)
-    latent.latent_append(ctx, y, a, w.inv_freq, places, cache, w.latent_norm, cfg.eps)
+    latent.latent_append(ctx, y, a, w.inv_freq, step.places, cache, w.latent_norm, cfg.eps)
+    n_single = step.n_single
     if n_single:
-        head_places = RowPlaces(None if places.slot is None else places.slot[:n_single], places.pos[:n_single])
-        _attend_rows(ctx, state, i, _sub(y, 0, n_single), _sub(z, 0, n_single, 0, a.heads * a.vdim), head_places, span)
-    if plans:
-        _attend_prompts(ctx, state, i, y, _sub(z, 0, T, 0, a.heads * a.vdim), plans[a.window])
+        _attend_rows(ctx, state, i, _sub(y, 0, n_single), _sub(z, 0, n_single, 0, a.heads * a.vdim), step.single_places(), step.span)
+    if step.plans:
+        _attend_prompts(ctx, state, i, y, _sub(z, 0, T, 0, a.heads * a.vdim), step.plans[a.window])
     linear(ctx, z, w.w_out, w.a_cols + w.ff_cols, [OutputSegment(cfg.width, SEG_F32, x)], residual=x)
     if lc.router:
         moe.moe_feed_forward(ctx, h, logits, w.experts, lc.router, _moe_scratch(state, lc, w, T), x)
@@ -385,137 +332,13 @@ def _attend_prompts(ctx, state: GigezenState, i: int, y: GPUBuffer2D, z: GPUBuff
                           cache, z)
 
 
-def _run(ctx, state: GigezenState, ids: torch.Tensor, places: RowPlaces, rows: int, n_single: int, span: int,
-         plans: Dict[int, PromptPlan], row_index: Optional[torch.Tensor], n_out: int) -> None:
-    """Embedding, all layers and, for the ``n_out`` rows of ``row_index`` (None: all), the logits."""
-    cfg, w = state.cfg, state.weights
-    x = state.rows("x", rows, cfg.width, torch.float32)
-    embedding_rows(ctx, w.embedding, ids, x)
-    for i in range(len(cfg.layers)):
-        _layer(ctx, state, i, x, places, n_single, span, plans)
-    if n_out == 0:
-        return
-    hl = state.rows("h_out", n_out, cfg.width, state.dtype)
-    rms_norm(ctx, x, w.final_norm, hl, cfg.eps, weight_offset=1.0, row_index=row_index)
-    out = state.rows("logits", n_out, cfg.vocab_size, torch.float32)
-    linear(ctx, hl, w.head, cfg.width, [OutputSegment(cfg.vocab_size, SEG_F32, out)])
-    state.logits = out
-
-
-def decode_step(ctx: GPUContext, state: GigezenState, token_ids: GPUBuffer1D, next_ids: Optional[GPUBuffer1D] = None) -> None:
-    """One new token for every sequence (``token_ids`` int32 ``[batch_size]``): positions come from the lengths on the device,
-    which advance behind the step, so the call can be captured into a graph (``model.GraphedDecodeStep``).  Logits (fp32) are
-    left in ``state.logits``, the greedy tokens in ``next_ids``.  Between ``batch_begin`` and ``batch_commit``."""
-    upper = state.caches[0].current_len
-    if upper >= state.max_seq_len:
-        raise ValueError(f"Cache is full: current_len={upper}, max_seq_len={state.max_seq_len}")
-    B = state.batch_size
-    _run(ctx, state, token_ids.buffer, RowPlaces(None, state.seq_lens), B, B, upper + 1, {}, None, B)
-    if next_ids is not None:
-        argmax(ctx, state.logits, next_ids)
-    _check(_lib.b2kv_advance_lengths(state.seq_lens.data_ptr(), B, 1, batch_op_begin(ctx)))
-    state.lengths = [v + 1 for v in state.lengths]
-    for c in state.owned.values():
-        c.current_len += 1
-
-
-def forward(ctx: GPUContext, state: GigezenState, entries: Sequence[Tuple[int, Sequence[int], Sequence[int]]]) -> Optional[torch.Tensor]:
-    """One step over ``entries`` = (sequence, its next tokens, the places among them whose logits are wanted): appends the
-    tokens to their sequences and returns the wanted logits, fp32 ``[wanted, vocab]`` in the order asked for (None if none).
-    Opens and commits a batch of its own."""
-    seen = set()
-    for slot, tokens, _ in entries:
-        if not 0 <= slot < state.batch_size or slot in seen:
-            raise ValueError(f"sequence {slot} is out of range or appears twice in a step")
-        seen.add(slot)
-        if len(tokens) == 0:
-            raise ValueError("an entry needs at least one token")
-        if state.lengths[slot] + len(tokens) > state.max_seq_len:
-            raise ValueError(f"Cache is full: current_len={state.lengths[slot]} + {len(tokens)}, max_seq_len={state.max_seq_len}")
-    short = [len(t) <= SHORT_ENTRY or not state.prompt_form for _, t, _ in entries]
-    order = sorted(range(len(entries)), key=lambda j: not short[j])  # stable: short entries first
-    ids, slots, pos, first_row, spans, lens = [], [], [], {}, [], list(state.lengths)
-    T, n_single, span = 0, 0, 1
-    for j in order:
-        slot, tokens, _ = entries[j]
-        first_row[j] = T
-        start, n = lens[slot], len(tokens)
-        if short[j]:
-            n_single += n
-            span = max(span, start + n)
-        else:
-            spans.append((T, n, slot, start))
-        ids.append(np.asarray(tokens, dtype=np.int32))
-        slots.append(np.full(n, slot, dtype=np.int32))
-        pos.append(np.arange(start, start + n, dtype=np.int32))
-        T += n
-        lens[slot] = start + n
-    want = [first_row[j] + int(p) for j in range(len(entries)) for p in entries[j][2]]
-    n_out = len(want)
-    windows = sorted({lc.attention.window for lc in state.cfg.layers}) if spans else []
-    plans = {win: PromptPlan.build(spans, win, state.max_seq_len) for win in windows}
-    # one upload per step: ids, sequences, positions, wanted rows, lengths behind the step, prompt tables
-    parts = [np.concatenate(ids), np.concatenate(slots), np.concatenate(pos), want, lens] + [plans[win].rows() for win in windows]
-    host = torch.from_numpy(np.concatenate([np.asarray(part, dtype=np.int32) for part in parts])).pin_memory()
-    pieces = list(host.to(ctx.device, non_blocking=True).split([len(part) for part in parts]))
-    for win, table in zip(windows, pieces[5:]):
-        plans[win].table = table
-    batch_begin(ctx)
-    _run(ctx, state, pieces[0], RowPlaces(pieces[1], pieces[2]), T, n_single, span, plans, pieces[3], n_out)
-    batch_commit(ctx)
-    state.seq_lens.copy_(pieces[4])
-    state.lengths = lens
-    state._sync_upper_bound()
-    return state.logits.buffer if n_out else None
-
-
 # ---------------------------------------------------------------------------------------------------------------
 # the served model
 # ---------------------------------------------------------------------------------------------------------------
 
-class _Lengths:
-    """What ``generate_text`` resets before a generation: every sequence at once."""
-
-    seq_lens = None
-
-    def __init__(self, state: GigezenState):
-        self.state = state
-
-    @property
-    def current_len(self) -> int:
-        return max(self.state.lengths)
-
-    @current_len.setter
-    def current_len(self, value: int) -> None:
-        state_set_lengths(self.state, [value] * self.state.batch_size)
-
-
-class GigezenModel:
-    """The registry's face of the design: the interface ``generate_text`` drives (on sequence 0), and steps over any mix of
-    sequences and portions."""
-
-    def __init__(self, ctx: GPUContext, cfg: GigezenConfig, weights: GigezenWeights, dtype: torch.dtype, batch_size: int,
-                 max_tokens: int):
-        self.ctx, self.cfg = ctx, cfg
-        self.state = state_create(ctx, cfg, weights, batch_size, max_tokens, dtype)
-        self.context, self.vocab_size = max_tokens, cfg.vocab_size
-        self.cache = _Lengths(self.state)
-
-    def forward(self, entries) -> Optional[torch.Tensor]:
-        return forward(self.ctx, self.state, entries)
-
-    def release(self, slot: int) -> None:
-        state_release(self.state, slot)
-
-    def prefill(self, tokens: Sequence[int]) -> torch.Tensor:
-        return self.forward([(0, list(tokens), [len(tokens) - 1])])
-
-    def decode_step(self, token: int) -> torch.Tensor:
-        return self.forward([(0, [int(token)], [0])])
-
-
 @register_model("Gigezen")
 def _build(ctx: GPUContext, config: dict, weights: Dict[str, torch.Tensor], dtype: torch.dtype, batch_size: int,
-           max_tokens: int) -> GigezenModel:
+           max_tokens: int) -> ServedModel:
     cfg = GigezenConfig.from_json(config)
-    return GigezenModel(ctx, cfg, prepare_weights(ctx, cfg, weights, dtype), dtype, batch_size, max_tokens)
+    return ServedModel(ctx, state_create(ctx, cfg, prepare_weights(ctx, cfg, weights, dtype), batch_size, max_tokens, dtype),
+                       cfg.vocab_size)

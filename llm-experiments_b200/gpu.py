@@ -21,6 +21,7 @@ from .buffers import (
     gpu_buffer_zerofy,
 )
 from .device import context_create, device_config_create, device_create, pipeline_cache_create
+from .gqa import gqa_append, gqa_decode, gqa_prefill
 from .kv_cache import (
     attention_with_kv_cache,
     kv_cache_create,
@@ -32,8 +33,9 @@ from .kv_cache import (
 from .latent import latent_append, latent_decode, latent_prefill
 from .moe import moe_feed_forward
 from .projection import linear, matmul, qkv_project_append
+from .recurrent import gated_linear_attention
 from .registry import architectures, load_model
-from .step_tail import argmax, embedding, embedding_rows, extract_last_tokens, layernorm, rms_norm, softmax
+from .step_tail import argmax, embedding, embedding_rows, extract_last_tokens, layernorm, layernorm_rows, rms_norm, softmax
 from .types import GPUBuffer1D, GPUBuffer2D, GPUConfig, GPUContext, KVCache, KVCacheConfig, KVCacheLayer
 
 __all__ = [
@@ -51,5 +53,6 @@ __all__ = [
     "qkv_project_append", "matmul",
     # extensions: building blocks of decoders with a 32-bit residual stream, and models from folders
     "linear", "embedding_rows", "rms_norm", "latent_append", "latent_decode", "latent_prefill", "moe_feed_forward",
+    "layernorm_rows", "gqa_append", "gqa_decode", "gqa_prefill", "gated_linear_attention",
     "architectures", "load_model",
 ]

@@ -104,12 +104,13 @@ class PromptPlan:
     BLOCK = 256  # query rows of one block of the kernel
 
     @staticmethod
-    def build(spans, window: int, max_seq_len: int) -> "PromptPlan":
-        """``spans``: (row0, n, sequence, start position); the table is filled in by ``rows()`` + an upload."""
+    def build(spans, window: int, max_seq_len: int, in_place: bool = False) -> "PromptPlan":
+        """``spans``: (row0, n, sequence, start position); the table is filled in by ``rows()`` + an upload.  ``in_place``: keys
+        and values are read from the cache itself, nothing is expanded."""
         portions, at, blocks = [], 0, 0
         for row0, n, slot, start in spans:
             lo = max(0, start - window + 1) if window > 0 else 0
-            portions.append((row0, n, slot * max_seq_len + lo, start + n - lo, at))
+            portions.append((row0, n, slot * max_seq_len + lo, start + n - lo, slot * max_seq_len + lo if in_place else at))
             at += start + n - lo
             blocks += (n + PromptPlan.BLOCK - 1) // PromptPlan.BLOCK
         return PromptPlan(portions=portions, table=None, n_blocks=blocks, kv_rows=at)

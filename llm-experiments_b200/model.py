@@ -251,6 +251,8 @@ class GraphedDecodeStep:
         if max(keep_len) >= cap:
             raise ValueError(f"Cache is full: current_len={max(keep_len)}, max_seq_len={cap}")
         keep_dev = [c.seq_lens.clone() for c in caches]
+        recurrent = list(getattr(state, "recurrent", {}).values())  # (the cache rows the warm-up writes are written again)
+        keep_rec = [t.clone() for t in recurrent]
         keep_tok = self.token_ids.buffer.clone()
         side = torch.cuda.Stream(device=ctx.device)
         side.wait_stream(torch.cuda.current_stream(ctx.device))
@@ -258,6 +260,8 @@ class GraphedDecodeStep:
             c.current_len = cap - 1
         with torch.cuda.stream(side):
             self._record()  # warm-up: nothing allocates or configures a kernel inside the capture
+            for t, kept in zip(recurrent, keep_rec):
+                t.copy_(kept)
             for c, n, dev in zip(caches, keep_len, keep_dev):
                 c.current_len = cap - 1  # launches sized for the longest sequence the cache can hold
                 c.seq_lens.copy_(dev)

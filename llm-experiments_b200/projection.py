@@ -17,10 +17,10 @@ from typing import Optional, Sequence
 import torch
 
 from . import _native
-from ._native import SEG_F32, SEG_GLU_CLAMP, SEG_GLU_SILU, SEG_STORE  # noqa: F401
+from ._native import SEG_F32, SEG_GLU_CLAMP, SEG_GLU_SILU, SEG_RELU2, SEG_SOFTCAP, SEG_STORE  # noqa: F401
 from .batch import batch_op_begin, dev_status_ptr, reference_op, validate_buffer_shape_2d
 from .kv_cache import _ptr, cache_strides, dtype_code
-from .types import GPUBuffer2D, GPUContext, KVCache
+from .types import GPUBuffer1D, GPUBuffer2D, GPUContext, KVCache
 
 
 @reference_op("matmul")
@@ -108,7 +108,8 @@ def qkv_project_append(ctx: GPUContext, cache: KVCache, layer_idx: int, x: GPUBu
 class OutputSegment:
     """Columns of a linear layer's weight up to ``end`` (from the end of the segment before) and where their products go:
     ``SEG_STORE`` in the storage type, ``SEG_F32`` in fp32 (with the residual added), ``SEG_GLU_SILU`` / ``SEG_GLU_CLAMP``
-    as gated pairs, (gate, up) in neighbouring columns, giving half as many output columns.  ``out`` may be a view of some
+    as gated pairs, (gate, up) in neighbouring columns, giving half as many output columns, ``SEG_RELU2`` as the square of the
+    positive part, ``SEG_SOFTCAP`` in fp32 squeezed into (-limit, limit) by a tanh.  ``out`` may be a view of some
     columns of a wider buffer; group g of a grouped product writes ``group`` elements further on per group."""
 
     end: int
@@ -120,8 +121,9 @@ class OutputSegment:
 @reference_op("linear")
 def linear(ctx: GPUContext, x: GPUBuffer2D, w: GPUBuffer2D, k: int, segments: Sequence[OutputSegment],
            residual: Optional[GPUBuffer2D] = None, limit: float = 0.0, groups: int = 1, group_x: int = 0, group_w: int = 0,
-           group_rows: Optional[torch.Tensor] = None, max_group_rows: int = 0, path: int = 0) -> None:
-    """``x @ w`` with the output columns cut into segments, fp32 or bfloat16 storage, any sizes (``b2kv_linear``).
+           group_rows: Optional[torch.Tensor] = None, max_group_rows: int = 0, path: int = 0,
+           bias: Optional[GPUBuffer1D] = None) -> None:
+    """``x @ w`` (``+ bias``, fp32) with the output columns cut into segments, fp32 or bfloat16 storage, any sizes (``b2kv_linear``).
 
     ``x`` ``[rows, >= k]`` and ``w`` (rows of the weight matrix, ``[in, out]``) may be views with a row pitch.  With
     ``groups`` > 1, group g reads ``x`` from element ``g * group_x`` on and ``w`` from ``g * group_w`` on (the heads of a
@@ -140,7 +142,7 @@ def linear(ctx: GPUContext, x: GPUBuffer2D, w: GPUBuffer2D, k: int, segments: Se
                            max_group_rows=max_group_rows, n_seg=len(segments), dtype=dtype_code(x.buffer.dtype), path=path,
                            limit=limit)
     for i, s in enumerate(segments):
-        want = torch.float32 if s.kind == SEG_F32 else x.buffer.dtype
+        want = torch.float32 if s.kind in (SEG_F32, SEG_SOFTCAP) else x.buffer.dtype
         if s.out.buffer.dtype != want or s.out.buffer.stride(1) != 1 or s.out.shape[0] < rows:
             raise ValueError(f"linear: output of segment {i} must be {want} with at least {rows} rows of contiguous elements")
         a.seg[i] = _native.Segment(out=s.out.buffer.data_ptr(), ld=s.out.buffer.stride(0), group=s.group, end=s.end,
@@ -149,6 +151,10 @@ def linear(ctx: GPUContext, x: GPUBuffer2D, w: GPUBuffer2D, k: int, segments: Se
         if residual.buffer.dtype != torch.float32:
             raise ValueError("linear: the residual must be float32")
         a.residual, a.ld_residual = residual.buffer.data_ptr(), residual.buffer.stride(0)
+    if bias is not None:
+        if bias.buffer.dtype != torch.float32 or bias.size < n:
+            raise ValueError(f"linear: the bias must be {n} float32 values")
+        a.bias = bias.buffer.data_ptr()
     if group_rows is not None:
         a.group_rows = group_rows.data_ptr()
     stream = batch_op_begin(ctx)

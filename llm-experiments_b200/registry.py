@@ -31,7 +31,7 @@ def architectures():
 
 
 def _import_models() -> None:
-    from . import gigezen, model  # noqa: F401  (they register themselves)
+    from . import bamasun, gigezen, model  # noqa: F401  (they register themselves)
 
 
 def build_model(ctx: GPUContext, config: dict, weights: Dict[str, torch.Tensor], dtype: torch.dtype = torch.bfloat16,

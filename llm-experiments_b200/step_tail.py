@@ -93,14 +93,40 @@ def layernorm(ctx: GPUContext, input_buf: GPUBuffer2D, gamma: GPUBuffer1D, beta:
 
 
 @reference_op("embedding")
-def embedding_rows(ctx: GPUContext, table: GPUBuffer2D, ids: torch.Tensor, output: GPUBuffer2D) -> None:
-    """``output[i] = table[ids[i]]`` as fp32 rows, no position added: the start of a 32-bit residual stream."""
+def embedding_rows(ctx: GPUContext, table: GPUBuffer2D, ids: torch.Tensor, output: GPUBuffer2D, scale: float = 1.0,
+                   copy: GPUBuffer2D = None) -> None:
+    """``output[i] = table[ids[i]] * scale`` as fp32 rows, no position added: the start of a 32-bit residual stream.  ``copy`` gets
+    the same rows in the table's type."""
     rows, dim = output.shape
     if table.shape[1] != dim or ids.numel() < rows or ids.dtype != torch.int32:
         raise ValueError("embedding_rows needs one int32 id per output row and a table of the output's width")
+    if copy is not None and (copy.shape != output.shape or copy.buffer.dtype != table.buffer.dtype or not copy.buffer.is_contiguous()):
+        raise ValueError("embedding_rows: the copy must be contiguous rows of the output's shape in the table's type")
     stream = batch_op_begin(ctx)
-    _native.check(_native.lib.b2kv_embed_rows(table.buffer.data_ptr(), ids.data_ptr(), _f32(output, "output"), rows, dim,
+    _native.check(_native.lib.b2kv_embed_rows(table.buffer.data_ptr(), ids.data_ptr(), _f32(output, "output"),
+                                              None if copy is None else copy.buffer.data_ptr(), scale, rows, dim,
                                               table.shape[0], _DTYPE_CODES[table.buffer.dtype], dev_status_ptr(ctx), stream))
+
+
+@reference_op("layernorm")
+def layernorm_rows(ctx: GPUContext, y: GPUBuffer2D, weight: GPUBuffer1D, bias: GPUBuffer1D, eps: float, x: GPUBuffer2D = None,
+                   output: GPUBuffer2D = None, row_index: torch.Tensor = None) -> None:
+    """Layer norm of the fp32 rows ``y[r]``, ``r = row_index[i]`` (or ``i``).  With ``x`` (fp32) the normed rows are added to it;
+    ``output`` (float32 or bfloat16) gets the new rows of ``x``, or without ``x`` the normed rows."""
+    if x is None and output is None:
+        raise ValueError("layernorm_rows needs x or output")
+    rows, size = (output if x is None else x).shape
+    validate_buffer_shape_1d(weight, size, "weight")
+    validate_buffer_shape_1d(bias, size, "bias")
+    if y.shape[1] != size or (row_index is None and y.shape[0] < rows) or (output is not None and output.shape != (rows, size)):
+        raise ValueError(f"layernorm_rows shape mismatch: y {tuple(y.shape)}, rows {rows} x {size}")
+    stream = batch_op_begin(ctx)
+    ptr = lambda b: None if b is None else b.buffer.data_ptr()  # noqa: E731
+    ld = lambda b: 0 if b is None else b.buffer.stride(0)  # noqa: E731
+    dt = _DTYPE_CODES[torch.float32 if output is None else output.buffer.dtype]
+    _native.check(_native.lib.b2kv_layernorm_rows(ptr(y), ld(y), None if row_index is None else row_index.data_ptr(),
+                                                  _f32(weight, "weight"), _f32(bias, "bias"), ptr(x), ld(x), ptr(output), ld(output),
+                                                  rows, size, eps, dt, stream))
 
 
 @reference_op("rms_norm")

@@ -112,8 +112,8 @@ def test_safetensors_round_trip_and_damage(pkg, tmp_path):
 def test_registry_knows_the_models_and_says_so(pkg):
     from llm_experiments_b200 import registry
 
-    assert registry.architectures() == ["GPTDecoder", "Gigezen"]
-    with pytest.raises(ValueError, match="GPTDecoder, Gigezen"):
+    assert registry.architectures() == ["Bamasun", "GPTDecoder", "Gigezen"]
+    with pytest.raises(ValueError, match="Bamasun, GPTDecoder, Gigezen"):
         registry.build_model(None, {"architecture": "none"}, {})
 
 
