@@ -36,6 +36,7 @@ static Knob g_knobs[] = {
     {"matmul_splits", 0},  // ranges of input features per tile in b2kv_matmul_rows (0 = by shape)
     {"decode_dynamic_chunks", 0},  // small chunks of the decode's token space handed out on demand: 0 = by size, 1 = always, 2 = never
     {"serial_launches", 0},  // 1 = no kernel is launched ahead of the end of the kernel before it (plain stream order)
+    {"gqa_decode_share", 0},  // 128-key tiles per share in b2kv_gqa_decode (0 = by size)
     {"gemm_variant", 0},   // b2kv_matmul: 0 = by shape and device, 1 = one CTA per tile, 2 / 3 = CTA pairs, 64 / 128 features per stage
 };
 
