@@ -109,6 +109,21 @@ WORKLOADS = {
     "gigezen_prefill_small": dict(kind="gigezen", phase="prefill", B=2, N=2048, width=2048, heads=16, ff=5440, layers=2, experts=64,
                                   top=6, expert_ff=1408, window=1024, vocab=32768,
                                   desc="prompts of B=2 x N=2048 tokens through 2 layers of a width-2048 Gigezen model, window 1024"),
+    "bamasun_decode": dict(kind="bamasun", phase="decode", B=64, lo=512, hi=8192, width=4096, heads=32, kv_heads=8, gla_heads=16,
+                           ff=16384, layers=4, vocab=32768, dtype_text="bf16 operands, fp32 accumulation, residual, norms, scores and state",
+                           desc="one cached decode step of a 4-layer Bamasun model (width 4096; attention of 32 heads on 8 key / value heads "
+                                "of 128 and gated linear attention of 16 heads of 128 x 256 in turn; feed-forward 16384; the second attention "
+                                "layer reads the first one's keys): B=64, len~U[512,8192] seed 0"),
+    "bamasun_decode_small": dict(kind="bamasun", phase="decode", B=8, lo=128, hi=1024, width=2048, heads=16, kv_heads=4, gla_heads=8,
+                                 ff=8192, layers=4, vocab=32768, dtype_text="bf16 operands, fp32 accumulation, residual, norms, scores and state",
+                                 desc="one cached decode step of a 4-layer Bamasun model of width 2048: B=8, len~U[128,1024]"),
+    "bamasun_prefill": dict(kind="bamasun", phase="prefill", B=8, N=4096, width=4096, heads=32, kv_heads=8, gla_heads=16, ff=16384,
+                            layers=2, vocab=32768, dtype_text="bf16 operands, fp32 accumulation, residual, norms, scores and state",
+                            desc="prompts of B=8 x N=4096 tokens through 2 layers (one of attention, one recurrent) of the width-4096 "
+                                 "Bamasun model"),
+    "bamasun_prefill_small": dict(kind="bamasun", phase="prefill", B=2, N=2048, width=2048, heads=16, kv_heads=4, gla_heads=8, ff=8192,
+                                  layers=2, vocab=32768, dtype_text="bf16 operands, fp32 accumulation, residual, norms, scores and state",
+                                  desc="prompts of B=2 x N=2048 tokens through 2 layers of a width-2048 Bamasun model"),
 }
 SLACK = 1024  # rows of head-room above the longest sequence for the appended tokens
 
@@ -1070,115 +1085,110 @@ def gigezen_config(w):
     return dict(architecture="Gigezen", layers=layers, vocab=w["vocab"], width=w["width"], norm=dict(eps=1e-6))
 
 
-def run_gigezen(h: Harness, w):
-    """A Gigezen model with random weights: a whole decode step (generated tokens/s, HBM roofline over every weight once and the
-    latents attended) or whole prompts (prompt tokens/s, tensor roofline), and every kernel of the design timed alone on the
-    model's own buffers, each with its roofline.  Those of a decode step are timed ten at a time in a graph; kernels whose operands fit L2 say so."""
-    torch, gpu, ctx = h.torch, h.gpu, h.ctx
-    from llm_experiments_b200 import gigezen, latent, moe
-    from llm_experiments_b200.model import GraphedDecodeStep
-    from llm_experiments_b200.projection import SEG_F32, SEG_GLU_CLAMP, SEG_GLU_SILU, SEG_STORE, OutputSegment, linear
+class ServedRun:
+    """What the benchmarks of served designs share: a state with random cache contents, a whole decode step (eager, end to end, as a
+    replayed graph) or whole prompts, and kernels timed alone."""
 
-    world, device, decode = h.world, h.device, w["phase"] == "decode"
-    cfg_json = gigezen_config(w)
-    cfg = gigezen.GigezenConfig.from_json(cfg_json)
-    weights = gigezen.prepare_weights(ctx, cfg, gigezen.random_tensors(ctx, cfg_json, seed=7000 + h.rank), torch.bfloat16)
-    h.release()
-    B, width, H, V = w["B"], w["width"], w["heads"], w["vocab"]
-    T_max = (w["hi"] if decode else w["N"]) + 8
-    state = gigezen.state_create(ctx, cfg, weights, B, T_max)
-    gen = torch.Generator(device=device).manual_seed(7100 + h.rank)
-    for c in state.caches:
-        c.layers[0].k_cache.buffer.normal_(generator=gen)
-        c.layers[0].v_cache.buffer.normal_(generator=gen)
-    peak, sustained, burst, kind = measured_peaks()
-    a, dense_w, mix_w = cfg.layers[0].attention, weights.layers[0], weights.layers[1]
-    router = cfg.layers[1].router
-    per_head = H * (a.dim + a.vdim) * a.kv_rank  # key and value matrices
-    dense_params = width * (H * (a.dim + a.rot) + a.kv_rank + a.rot) + per_head + width * H * a.vdim + 3 * width * w["ff"]
-    attn_params = width * H * (a.dim + a.rot) + per_head + width * H * a.vdim
-    expert_params = 3 * width * w["expert_ff"]
-    n_dense, n_mix = (w["layers"] + 1) // 2, w["layers"] // 2
+    def __init__(self, h: "Harness", w, state, T_max):
+        self.h, self.w, self.state, self.decode = h, w, state, w["phase"] == "decode"
+        self.kernels = []
+        torch, gpu, ctx, device = h.torch, h.gpu, h.ctx, h.device
+        from llm_experiments_b200 import serving
 
-    if decode:
-        lens = make_lengths(w)
-        gigezen.state_set_lengths(state, lens)
-        lens_dev, lens_list = state.seq_lens.clone(), [int(v) for v in lens]
-        tok_b = h.wrap1(torch.randint(0, V, (B,), generator=gen, device=device, dtype=torch.int32))
-        next_b = h.wrap1(torch.empty(B, dtype=torch.int32, device=device))
-        tok_h, next_h = tok_b.buffer.cpu().pin_memory(), torch.empty(B, dtype=torch.int32).pin_memory()
+        self.serving = serving
+        gen = torch.Generator(device=device).manual_seed(7100 + h.rank)
+        for c in state.owned.values():
+            c.layers[0].k_cache.buffer.normal_(generator=gen)
+            c.layers[0].v_cache.buffer.normal_(generator=gen)
+        B, V = w["B"], w["vocab"]
+        if self.decode:
+            self.lens = make_lengths(w)
+            serving.state_set_lengths(state, self.lens)
+            self.lens_dev, self.lens_list = state.seq_lens.clone(), [int(v) for v in self.lens]
+            self.tok_b = h.wrap1(torch.randint(0, V, (B,), generator=gen, device=device, dtype=torch.int32))
+            self.next_b = h.wrap1(torch.empty(B, dtype=torch.int32, device=device))
+            self.tok_h, self.next_h = self.tok_b.buffer.cpu().pin_memory(), torch.empty(B, dtype=torch.int32).pin_memory()
+            self.rows, self.h2d, self.d2h = B, B * 4, B * 4
+        else:
+            N = w["N"]
+            prompts = [np.random.default_rng(s).integers(0, V, size=N).astype(np.int32) for s in range(B)]
+            self.out_h = torch.empty((B, V), dtype=torch.float32).pin_memory()
+            self.entries = [(b, prompts[b], [N - 1]) for b in range(B)]
+            self.rows, self.h2d, self.d2h = B * N, 3 * B * N * 4, B * V * 4
+        self.rnd = torch.Generator(device=device).manual_seed(5)
 
-        def rewind():
-            state.seq_lens.copy_(lens_dev)
-            state.lengths = list(lens_list)
-            for c in state.caches:
-                c.current_len = max(lens_list)
+    def rewind(self):
+        self.state.seq_lens.copy_(self.lens_dev)
+        self.state.lengths = list(self.lens_list)
+        for c in self.state.caches:
+            c.current_len = max(self.lens_list)
 
-        def step_device():
-            rewind()
-            gpu.batch_begin(ctx)
-            gigezen.decode_step(ctx, state, tok_b, next_b)
-            gpu.batch_commit(ctx)
+    def step_device(self):
+        h, state = self.h, self.state
+        if self.decode:
+            self.rewind()
+            h.gpu.batch_begin(h.ctx)
+            self.serving.decode_step(h.ctx, state, self.tok_b, self.next_b)
+            h.gpu.batch_commit(h.ctx)
+        else:
+            self.serving.state_reset(state)
+            self.serving.forward(h.ctx, state, self.entries)
 
-        def step_e2e():
-            gpu.gpu_buffer_1d_write(ctx, tok_h, tok_b)
-            step_device()
-            gpu.gpu_buffer_1d_read(ctx, next_b, next_h)
+    def step_e2e(self):
+        h = self.h
+        if self.decode:
+            h.gpu.gpu_buffer_1d_write(h.ctx, self.tok_h, self.tok_b)
+            self.step_device()
+            h.gpu.gpu_buffer_1d_read(h.ctx, self.next_b, self.next_h)
+        else:
+            self.step_device()
+            self.out_h.copy_(self.state.logits.buffer, non_blocking=True)
+            h.torch.cuda.current_stream().synchronize()
 
-        rows, tokens, h2d, d2h = B, B, B * 4, B * 4
-    else:
-        N = w["N"]
-        prompts = [np.random.default_rng(s).integers(0, V, size=N).astype(np.int32) for s in range(B)]
-        out_h = torch.empty((B, V), dtype=torch.float32).pin_memory()
-        entries = [(b, prompts[b], [N - 1]) for b in range(B)]
+    def measure(self):
+        """(steps, device-timed step, end-to-end step, graph record or None)."""
+        h, graph = self.h, None
+        steps = h.steps if self.decode else min(h.steps, 10)
+        m_step = h.measure(self.step_device, steps=steps)
+        m_e2e = h.measure(self.step_e2e, steps=max(2, min(steps, 20)), warmup=1, repeats=min(h.repeats, 3))
+        if self.decode:
+            from llm_experiments_b200.model import GraphedDecodeStep
 
-        def step_device():
-            gigezen.state_reset(state)
-            gigezen.forward(ctx, state, entries)
+            graphed = GraphedDecodeStep(h.ctx, self.state, step_fn=self.serving.decode_step)
+            self.rewind()
+            graphed.capture()
 
-        def step_e2e():
-            step_device()
-            out_h.copy_(state.logits.buffer, non_blocking=True)
-            torch.cuda.current_stream().synchronize()
+            def step_graph():
+                self.rewind()
+                graphed.step()
 
-        rows, tokens, h2d, d2h = B * N, B * N, 3 * B * N * 4, B * V * 4
+            m_graph = h.measure(step_graph)
+            graph = {"value": h.world * self.w["B"] / (m_graph["ms"] * 1e-3), "unit": "tokens/s", **spread(m_graph)}
+            self.rewind()
+        h.ctx.config.max_batch_operations = 10 ** 9
+        return steps, m_step, m_e2e, graph
 
-    sampler = h.sampler()
-    steps = h.steps if decode else min(h.steps, 10)
-    m_step = h.measure(step_device, steps=steps)
-    m_e2e = h.measure(step_e2e, steps=max(2, min(steps, 20)), warmup=1, repeats=min(h.repeats, 3))
-    graph = None
-    if decode:
-        graphed = GraphedDecodeStep(ctx, state, step_fn=gigezen.decode_step)
-        rewind()
-        graphed.capture()
+    def bf(self, r, c):
+        torch = self.h.torch
+        return self.h.wrap(torch.randn((r, c), generator=self.rnd, device=self.h.device).to(torch.bfloat16))
 
-        def step_graph():
-            rewind()
-            graphed.step()
+    def f32(self, r, c):
+        return self.h.wrap(self.h.torch.randn((r, c), generator=self.rnd, device=self.h.device))
 
-        m_graph = h.measure(step_graph)
-        graph = {"value": world * B / (m_graph["ms"] * 1e-3), "unit": "tokens/s", **spread(m_graph)}
-        rewind()
+    def view(self, b, c0, n):
+        return self.h.wrap(b.buffer[:, c0:c0 + n])
 
-    # ---- every kernel alone, on the rows, weights and cache of the step above
-    ctx.config.max_batch_operations = 10 ** 9
-    g = torch.Generator(device=device).manual_seed(5)
-    bf = lambda r, c: h.wrap(torch.randn((r, c), generator=g, device=device).to(torch.bfloat16))  # noqa: E731
-    f32 = lambda r, c: h.wrap(torch.randn((r, c), generator=g, device=device))  # noqa: E731
-    view = lambda b, c0, n: h.wrap(b.buffer[:, c0:c0 + n])  # noqa: E731
-    x, hb = f32(rows, width), bf(rows, width)
-    y, z = bf(rows, dense_w.y_cols), bf(rows, dense_w.a_cols + dense_w.ff_cols)
-    cache = state.caches[0]
-    kernels = []
+    def kernel(self, name, fn, flops=0, nbytes=0, note=None):
+        """Times fn alone: those of a decode step ten at a time in a graph (a launch from Python takes longer than most)."""
+        h, torch = self.h, self.h.torch
+        peak, sustained, _, _ = measured_peaks()
 
-    def kernel(name, fn, flops=0, nbytes=0, note=None):
         def once():
-            gpu.batch_begin(ctx)
+            h.gpu.batch_begin(h.ctx)
             fn()
-            gpu.batch_commit(ctx)
+            h.gpu.batch_commit(h.ctx)
 
-        if decode:  # ten launches in a graph: a launch from Python takes longer than most of these kernels
+        if self.decode:
             side = torch.cuda.Stream()
             side.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(side):
@@ -1188,15 +1198,75 @@ def run_gigezen(h: Harness, w):
                     for _ in range(10):
                         once()
             torch.cuda.current_stream().wait_stream(side)
-            m = h.measure(graph_k.replay, steps=10, repeats=3)
-            t = m["ms"] * 1e-4
+            t = h.measure(graph_k.replay, steps=10, repeats=3)["ms"] * 1e-4
         else:
-            m = h.measure(once, steps=10, repeats=3)
-            t = m["ms"] * 1e-3
+            t = h.measure(once, steps=10, repeats=3)["ms"] * 1e-3
         need_t, need_b = flops / (sustained * 1e12), nbytes / (peak * 1e9)
-        kernels.append({"kernel": name, "us": 1e6 * t, "bound": "tensor" if need_t > need_b else "hbm",
-                        "frac": max(need_t, need_b) / t, "TFLOP/s": flops / t / 1e12, "GB/s": nbytes / t / 1e9, **({"note": note} if note else {})})
+        self.kernels.append({"kernel": name, "us": 1e6 * t, "bound": "tensor" if need_t > need_b else "hbm", "frac": max(need_t, need_b) / t,
+                             "TFLOP/s": flops / t / 1e12, "GB/s": nbytes / t / 1e9, **({"note": note} if note else {})})
 
+    def record(self, measured, launches, clocks, nbytes, flops, **extra):
+        """The workload's line: whole step against its bytes (decoding) or flops (prompts)."""
+        h, w = self.h, self.w
+        steps, m_step, m_e2e, graph = measured
+        peak, sustained, _, kind = measured_peaks()
+        if self.decode:
+            bound, achieved, peak_v, unit = "hbm", nbytes / (m_step["ms"] * 1e-3) / 1e9, peak, "GB/s"
+            extra["algorithmic_bytes_per_launch"] = nbytes
+        else:
+            bound, achieved, peak_v, unit = "tensor", flops / (m_step["ms"] * 1e-3) / 1e12, sustained, "TFLOP/s"
+            extra["algorithmic_flops_per_launch"] = flops
+        status = int(h.ctx.dev_status.item()) if h.ctx.dev_status is not None else 0
+        tokens = h.world * self.rows
+        return {
+            "metric": "generated tokens/s (whole cached decode step of the model)" if self.decode else "prompt tokens/s (whole model)",
+            "value": tokens / (m_step["ms"] * 1e-3), "unit": "tokens/s", **spread(m_step), "steps": steps, "scaling": "weak",
+            "dtype": w.get("dtype_text", "bf16 operands, fp32 accumulation, residual, norms, scores and router"),
+            "config": {"workload": w["desc"], "batch_per_gpu": w["B"], "global_batch": h.world * w["B"],
+                       "l2": "weights and caches far larger than L2, no flush", "parallelism": f"batch-sharded x{h.world}, no collective"},
+            "e2e": {"value": tokens / (m_e2e["ms"] * 1e-3), "unit": "tokens/s", **spread(m_e2e), "h2d_bytes_per_step": self.h2d,
+                    "d2h_bytes_per_step": self.d2h},
+            "gpu_launches": steps * h.repeats * launches, "gpu_launches_per_step": launches, "clocks": clocks, "dev_status": status,
+            "cuda_graph": graph, "kernels": self.kernels,
+            "roofline": {"bound": bound, "kernel": "the step's kernels together", "achieved": achieved, "peak": peak_v, "unit": unit,
+                         "frac": achieved / peak_v, "peak_kind": kind, "traffic": None, **extra},
+        }
+
+
+def run_gigezen(h: Harness, w):
+    """A Gigezen model with random weights: a whole decode step (generated tokens/s, HBM roofline over every weight once and the
+    latents attended) or whole prompts (prompt tokens/s, tensor roofline), and every kernel of the design timed alone on the
+    model's own buffers, each with its roofline.  Those of a decode step are timed ten at a time in a graph; kernels whose operands fit L2 say so."""
+    torch, gpu, ctx = h.torch, h.gpu, h.ctx
+    from llm_experiments_b200 import gigezen, latent, moe
+    from llm_experiments_b200.projection import SEG_F32, SEG_GLU_CLAMP, SEG_GLU_SILU, SEG_STORE, OutputSegment, linear
+
+    device, decode = h.device, w["phase"] == "decode"
+    cfg_json = gigezen_config(w)
+    cfg = gigezen.GigezenConfig.from_json(cfg_json)
+    weights = gigezen.prepare_weights(ctx, cfg, gigezen.random_tensors(ctx, cfg_json, seed=7000 + h.rank), torch.bfloat16)
+    h.release()
+    B, width, H, V = w["B"], w["width"], w["heads"], w["vocab"]
+    T_max = (w["hi"] if decode else w["N"]) + 8
+    state = gigezen.state_create(ctx, cfg, weights, B, T_max)
+    run = ServedRun(h, w, state, T_max)
+    a, dense_w, mix_w = cfg.layers[0].attention, weights.layers[0], weights.layers[1]
+    router = cfg.layers[1].router
+    per_head = H * (a.dim + a.vdim) * a.kv_rank  # key and value matrices
+    dense_params = width * (H * (a.dim + a.rot) + a.kv_rank + a.rot) + per_head + width * H * a.vdim + 3 * width * w["ff"]
+    attn_params = width * H * (a.dim + a.rot) + per_head + width * H * a.vdim
+    expert_params = 3 * width * w["expert_ff"]
+    n_dense, n_mix = (w["layers"] + 1) // 2, w["layers"] // 2
+
+    sampler = h.sampler()
+    measured = run.measure()
+    rows = run.rows
+
+    # ---- every kernel alone, on the rows, weights and cache of the step above
+    bf, f32, view, kernel = run.bf, run.f32, run.view, run.kernel
+    x, hb = f32(rows, width), bf(rows, width)
+    y, z = bf(rows, dense_w.y_cols), bf(rows, dense_w.a_cols + dense_w.ff_cols)
+    cache = state.caches[0]
     n_in, n_out = dense_w.y_cols + 2 * dense_w.ff_cols, dense_w.a_cols + dense_w.ff_cols
     kernel("rms_norm", lambda: gpu.rms_norm(ctx, x, dense_w.norm, hb, cfg.eps, weight_offset=1.0), 0, rows * width * 6)
     kernel("linear in (queries, latent, gated hidden rows)", lambda: linear(
@@ -1209,14 +1279,14 @@ def run_gigezen(h: Harness, w):
     if decode:
         places = latent.RowPlaces(None, state.seq_lens)
         ql, ol = bf(rows, H * a.kv_rank), bf(rows, H * a.kv_rank)
-        seen = int(np.minimum(lens + 1, w["window"]).sum())
+        seen = int(np.minimum(run.lens + 1, w["window"]).sum())
         kernel("latent_append", lambda: latent.latent_append(ctx, y, a, dense_w.inv_freq, places, cache, dense_w.latent_norm, cfg.eps), 0,
                rows * 2 * (2 * dense_w.y_cols + a.kv_rank + a.rot), "latency: a few hundred KB")
         kernel("linear per head (queries into the latent space)", lambda: linear(
             ctx, y, dense_w.key_absorb, a.dim, [OutputSegment(a.kv_rank, SEG_STORE, ql, group=a.kv_rank)], groups=H,
             group_x=a.dim + a.rot, group_w=a.dim * a.kv_rank), 2.0 * rows * H * a.dim * a.kv_rank,
             2 * (H * a.dim * a.kv_rank + rows * H * (a.dim + a.kv_rank)), "operands stay in L2 (one layer); latency-bound")
-        kernel("latent_decode", lambda: latent.latent_decode(ctx, ql, y, a, places, cache, ol, int(lens.max()) + 1),
+        kernel("latent_decode", lambda: latent.latent_decode(ctx, ql, y, a, places, cache, ol, int(run.lens.max()) + 1),
                2.0 * seen * H * (2 * a.kv_rank + a.rot), 2 * (seen * (a.kv_rank + a.rot) + 2 * rows * H * a.kv_rank))
         kernel("linear per head (values out of the latent space)", lambda: linear(
             ctx, ol, view(dense_w.expand, dense_w.k_cols, H * a.vdim), a.kv_rank,
@@ -1261,35 +1331,130 @@ def run_gigezen(h: Harness, w):
         2.0 * n_sel * width * e_ff, 2 * (used * width * e_ff + n_sel * (width + e_ff)))
     kernel("moe combine", lambda: moe.combine(ctx, x, router, scratch), 0, 2 * n_sel * width + 8 * rows * width)
     clocks = sampler.finish()
-    status = int(ctx.dev_status.item()) if ctx.dev_status is not None else 0
-
+    nbytes = flops = 0
+    extra = {}
     if decode:
         kv_bytes = w["layers"] * seen * 2 * (a.kv_rank + a.rot)
         weight_bytes = 2 * (n_dense * dense_params + n_mix * (attn_params + used * expert_params + width * router.experts) + width * V)
-        bound, achieved, peak_v, unit = "hbm", (kv_bytes + weight_bytes) / (m_step["ms"] * 1e-3) / 1e9, peak, "GB/s"
-        extra = {"algorithmic_bytes_per_launch": kv_bytes + weight_bytes, "kv_bytes": kv_bytes, "weight_bytes": weight_bytes}
+        nbytes, extra = kv_bytes + weight_bytes, {"kv_bytes": kv_bytes, "weight_bytes": weight_bytes}
     else:
         gemm = 2.0 * rows * (n_dense * dense_params + n_mix * (attn_params + router.top * expert_params))
         flops = gemm + w["layers"] * 2.0 * pairs * (a.dim + a.rot + a.vdim) + 2.0 * B * width * V
-        bound, achieved, peak_v, unit = "tensor", flops / (m_step["ms"] * 1e-3) / 1e12, sustained, "TFLOP/s"
-        extra = {"algorithmic_flops_per_launch": flops}
     launches = (9 * w["layers"] + 8 * n_mix + 5) if decode else ((6 + B) * w["layers"] + 8 * n_mix + 3)
-    return {
-        "metric": "generated tokens/s (whole cached decode step of the model)" if decode else "prompt tokens/s (whole model)",
-        "value": world * tokens / (m_step["ms"] * 1e-3), "unit": "tokens/s", **spread(m_step), "steps": steps, "scaling": "weak",
-        "dtype": "bf16 operands, fp32 accumulation, residual, norms, scores and router",
-        "config": {"workload": w["desc"], "batch_per_gpu": B, "global_batch": world * B,
-                   "l2": "weights and caches far larger than L2, no flush", "parallelism": f"batch-sharded x{world}, no collective"},
-        "e2e": {"value": world * tokens / (m_e2e["ms"] * 1e-3), "unit": "tokens/s", **spread(m_e2e), "h2d_bytes_per_step": h2d,
-                "d2h_bytes_per_step": d2h},
-        "gpu_launches": steps * h.repeats * launches, "gpu_launches_per_step": launches, "clocks": clocks, "dev_status": status,
-        "cuda_graph": graph, "kernels": kernels,
-        "roofline": {"bound": bound, "kernel": "the step's kernels together", "achieved": achieved, "peak": peak_v, "unit": unit,
-                     "frac": achieved / peak_v, "peak_kind": kind, "traffic": None, **extra},
-    }
+    return run.record(measured, launches, clocks, nbytes, flops, **extra)
 
 
-RUNNERS = {"gigezen": run_gigezen, "prefill": run_prefill, "qkv": run_qkv_append, "layer_step": run_decode_layer,
+def bamasun_config(w):
+    """config.json of the benchmark's model: attention and recurrent layers in turn; every second attention layer reads the keys
+    and values of the one before."""
+    layers, owner = [], None
+    for i in range(w["layers"]):
+        if i % 2 == 0:
+            mixer = dict(heads=w["heads"], kv_heads=w["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5, q_temp=dict(coef=0.1, every=1024))
+            if owner is None:
+                owner = i
+            else:
+                mixer["kv_from"], owner = owner, None
+            kind = "attention"
+        else:
+            mixer, kind = dict(heads=w["gla_heads"], dim=128, vdim=256, tau=16.0), "gla"
+        layers.append(dict(type=kind, mixer=mixer, mlp=dict(kind="dense", ff=w["ff"])))
+    return dict(architecture="Bamasun", layers=layers, vocab=w["vocab"], width=w["width"], norm=dict(eps=1e-6),
+                embedding=dict(scale=2.0), logit_softcap=30.0)
+
+
+def run_bamasun(h: Harness, w):
+    """A Bamasun model with random weights: a whole decode step (generated tokens/s, HBM roofline over every weight once, the keys
+    and values attended, the states read and written) or whole prompts (prompt tokens/s, tensor roofline), and every kernel of
+    the design timed alone on the model's own buffers."""
+    torch, gpu, ctx = h.torch, h.gpu, h.ctx
+    from llm_experiments_b200 import bamasun, gqa, latent, recurrent
+    from llm_experiments_b200.projection import SEG_F32, SEG_RELU2, SEG_SOFTCAP, SEG_STORE, OutputSegment, linear
+    from llm_experiments_b200.serving import RowSegments
+
+    device, decode = h.device, w["phase"] == "decode"
+    cfg_json = bamasun_config(w)
+    cfg = bamasun.BamasunConfig.from_json(cfg_json)
+    weights = bamasun.prepare_weights(ctx, cfg, bamasun.random_tensors(ctx, cfg_json, seed=7200 + h.rank), torch.bfloat16)
+    h.release()
+    B, width, V, ff = w["B"], w["width"], w["vocab"], w["ff"]
+    T_max = (w["hi"] if decode else w["N"]) + 8
+    state = bamasun.state_create(ctx, cfg, weights, B, T_max)
+    run = ServedRun(h, w, state, T_max)
+    sampler = h.sampler()
+    measured = run.measure()
+    rows, kernel, view, bf, f32 = run.rows, run.kernel, run.view, run.bf, run.f32
+
+    # ---- every kernel alone, on the rows, weights, caches and states of the step above
+    a, g, aw, gw = cfg.layers[0].attention, cfg.layers[1].gla, weights.layers[0], weights.layers[1]
+    nq, nkv = a.heads * a.dim, a.kv_heads * (a.dim + a.vdim)
+    gk, gv, rank = g.heads * g.dim, g.heads * g.vdim, 16
+    x, xb, yf = f32(rows, width), bf(rows, width), f32(rows, width)
+    ya, yg = bf(rows, aw.w_in.shape[1]), bf(rows, gw.w_in.shape[1])
+    oa, og, hid = bf(rows, aw.w_o.shape[0]), bf(rows, gw.w_o.shape[0]), bf(rows, ff)
+    zf = f32(rows, gw.w_a2.shape[1])
+    cache, rec = state.cache_of(0), state.recurrent[1]
+
+    def product(name, xin, wm, k, segments, n_real, out_bytes, **kw):
+        kernel(name, lambda: linear(ctx, xin, wm, k, segments, **kw), 2.0 * rows * k * n_real, 2 * (k * n_real + rows * k) + rows * out_bytes)
+
+    kernel("layer norm onto the residual", lambda: gpu.layernorm_rows(ctx, yf, aw.norm1.w, aw.norm1.b, cfg.eps, x=x, output=xb), 0,
+           rows * width * 14)
+    product("linear in, attention (q, k, v + bias)", xb, aw.w_in, width, [OutputSegment(ya.shape[1], SEG_STORE, ya)], nq + nkv,
+            2 * (nq + nkv), bias=aw.bias)
+    product("linear in, gla (q, k, v, gate, decay rows)", xb, gw.w_in, width, [OutputSegment(yg.shape[1], SEG_STORE, yg)],
+            2 * gk + 2 * gv + rank, 2 * (2 * gk + 2 * gv + rank))
+    decay_rows = view(yg, gw.cols[4], yg.shape[1] - gw.cols[4])
+    product("linear, decay logits (fp32)", decay_rows, gw.w_a2, gw.w_a2.shape[0], [OutputSegment(zf.shape[1], SEG_F32, zf)], gk, 4 * gk,
+            bias=gw.a2_bias)
+    product("linear out, attention (fp32)", oa, aw.w_o, oa.shape[1], [OutputSegment(width, SEG_F32, yf)], width, 4 * width)
+    product("linear up (squared relu)", xb, aw.w_up, width, [OutputSegment(ff, SEG_RELU2, hid)], ff, 2 * ff)
+    product("linear down (fp32)", hid, aw.w_down, ff, [OutputSegment(width, SEG_F32, yf)], width, 4 * width)
+    state_bytes = 8 * g.heads * g.dim * g.vdim  # read and written
+    gla_row = 2 * (2 * gk + 3 * gv) + 4 * gk
+    if decode:
+        places = latent.RowPlaces(None, state.seq_lens)
+        seen = int((run.lens + 1).sum())
+        kv_bytes = seen * 2 * nkv
+        kernel("gqa_append", lambda: gqa.gqa_append(ctx, ya, a, places, cache, True, aw.q_norm, aw.k_norm, cfg.eps), 0,
+               rows * 4 * (nq + nkv), "latency: a few hundred KB")
+        kernel("gqa_decode", lambda: gqa.gqa_decode(ctx, ya, a, aw.slopes, places, cache, oa, int(run.lens.max()) + 1),
+               2.0 * seen * a.heads * (a.dim + a.vdim), kv_bytes + rows * 2 * a.heads * (a.dim + a.vdim))
+        one = RowSegments(None, rows, 1)
+        kernel("gated linear attention, one token", lambda: recurrent.gated_linear_attention(
+            ctx, yg, gw.cols[:4], zf, g, gw.head_norm, cfg.eps, one, state.seq_lens, rec, og), 0, rows * (state_bytes + gla_row))
+        logits = f32(rows, V)
+        product("linear, logits (soft cap)", xb, weights.head, width, [OutputSegment(V, SEG_SOFTCAP, logits)], V, 4 * V, limit=30.0)
+    else:
+        N = w["N"]
+        pos = torch.arange(N, device=device, dtype=torch.int32).repeat(B)
+        places = latent.RowPlaces(torch.arange(B, device=device, dtype=torch.int32).repeat_interleave(N).contiguous(), pos)
+        plan = latent.PromptPlan.build([(b * N, N, b, 0) for b in range(B)], 0, T_max, in_place=True)
+        plan.table = torch.tensor(plan.rows(), dtype=torch.int32, device=device)
+        kernel("gqa_append", lambda: gqa.gqa_append(ctx, ya, a, places, cache, True, aw.q_norm, aw.k_norm, cfg.eps), 0, rows * 4 * (nq + nkv))
+        pairs = 0.5 * N * (N + 1) * B * a.heads
+        kernel("gqa_prefill", lambda: gqa.gqa_prefill(ctx, ya, a, aw.slopes, plan, cache, oa), 2.0 * pairs * (a.dim + a.vdim),
+               rows * 2 * (2 * nq + nkv))
+        table = torch.tensor([[b * N, N, b] for b in range(B)], dtype=torch.int32, device=device)
+        runs = RowSegments(table, B, N)
+        kernel("gated linear attention, prompts", lambda: recurrent.gated_linear_attention(
+            ctx, yg, gw.cols[:4], zf, g, gw.head_norm, cfg.eps, runs, pos, rec, og), 0, rows * gla_row + B * state_bytes,
+            "bytes: rows once; its products are not what bounds it")
+    clocks = sampler.finish()
+    mixers = [lc.attention is not None for lc in cfg.layers]
+    n_att, n_gla, n_own = sum(mixers), len(mixers) - sum(mixers), len(state.owned)
+    params = n_att * (width * nq + a.heads * a.vdim * width) + n_own * width * nkv + len(mixers) * 2 * width * ff + \
+        n_gla * (width * (2 * gk + 2 * gv + rank) + rank * gk + gv * width)
+    nbytes = flops = 0
+    if decode:
+        nbytes = n_att * kv_bytes + n_gla * rows * state_bytes + 2 * (params + width * V)
+    else:
+        flops = 2.0 * rows * params + n_att * 2.0 * pairs * (a.dim + a.vdim) + n_gla * 4.0 * rows * g.heads * g.dim * g.vdim + 2.0 * B * width * V
+    launches = 9 * n_att + 8 * n_gla + 5 if decode else 8 * (n_att + n_gla) + 3
+    return run.record(measured, launches, clocks, nbytes, flops)
+
+
+RUNNERS = {"gigezen": run_gigezen, "bamasun": run_bamasun, "prefill": run_prefill, "qkv": run_qkv_append, "layer_step": run_decode_layer,
            "prompt_layer": run_prompt_layer, "model_step": run_model_step}
 
 
