@@ -1369,7 +1369,7 @@ def run_bamasun(h: Harness, w):
     the design timed alone on the model's own buffers."""
     torch, gpu, ctx = h.torch, h.gpu, h.ctx
     from llm_experiments_b200 import bamasun, gqa, latent, recurrent
-    from llm_experiments_b200.projection import SEG_F32, SEG_RELU2, SEG_SOFTCAP, SEG_STORE, OutputSegment, linear
+    from llm_experiments_b200.projection import SEG_DECAY, SEG_F32, SEG_RELU2, SEG_SOFTCAP, SEG_STORE, OutputSegment, linear
     from llm_experiments_b200.serving import RowSegments
 
     device, decode = h.device, w["phase"] == "decode"
@@ -1392,7 +1392,7 @@ def run_bamasun(h: Harness, w):
     x, xb, yf = f32(rows, width), bf(rows, width), f32(rows, width)
     ya, yg = bf(rows, aw.w_in.shape[1]), bf(rows, gw.w_in.shape[1])
     oa, og, hid = bf(rows, aw.w_o.shape[0]), bf(rows, gw.w_o.shape[0]), bf(rows, ff)
-    zf = f32(rows, gw.w_a2.shape[1])
+    al = f32(rows, gw.w_a2.shape[1])
     cache, rec = state.cache_of(0), state.recurrent[1]
 
     def product(name, xin, wm, k, segments, n_real, out_bytes, **kw):
@@ -1405,8 +1405,8 @@ def run_bamasun(h: Harness, w):
     product("linear in, gla (q, k, v, gate, decay rows)", xb, gw.w_in, width, [OutputSegment(yg.shape[1], SEG_STORE, yg)],
             2 * gk + 2 * gv + rank, 2 * (2 * gk + 2 * gv + rank))
     decay_rows = view(yg, gw.cols[4], yg.shape[1] - gw.cols[4])
-    product("linear, decay logits (fp32)", decay_rows, gw.w_a2, gw.w_a2.shape[0], [OutputSegment(zf.shape[1], SEG_F32, zf)], gk, 4 * gk,
-            bias=gw.a2_bias)
+    product("linear, decays (fp32)", decay_rows, gw.w_a2, gw.w_a2.shape[0], [OutputSegment(al.shape[1], SEG_DECAY, al)], gk, 4 * gk,
+            limit=g.tau, bias=gw.a2_bias)
     product("linear out, attention (fp32)", oa, aw.w_o, oa.shape[1], [OutputSegment(width, SEG_F32, yf)], width, 4 * width)
     product("linear up (squared relu)", xb, aw.w_up, width, [OutputSegment(ff, SEG_RELU2, hid)], ff, 2 * ff)
     product("linear down (fp32)", hid, aw.w_down, ff, [OutputSegment(width, SEG_F32, yf)], width, 4 * width)
@@ -1422,7 +1422,7 @@ def run_bamasun(h: Harness, w):
                2.0 * seen * a.heads * (a.dim + a.vdim), kv_bytes + rows * 2 * a.heads * (a.dim + a.vdim))
         one = RowSegments(None, rows, 1)
         kernel("gated linear attention, one token", lambda: recurrent.gated_linear_attention(
-            ctx, yg, gw.cols[:4], zf, g, gw.head_norm, cfg.eps, one, state.seq_lens, rec, og), 0, rows * (state_bytes + gla_row))
+            ctx, yg, gw.cols[:4], al, g, gw.head_norm, cfg.eps, one, state.seq_lens, rec, og), 0, rows * (state_bytes + gla_row))
         logits = f32(rows, V)
         product("linear, logits (soft cap)", xb, weights.head, width, [OutputSegment(V, SEG_SOFTCAP, logits)], V, 4 * V, limit=30.0)
     else:
@@ -1438,7 +1438,7 @@ def run_bamasun(h: Harness, w):
         table = torch.tensor([[b * N, N, b] for b in range(B)], dtype=torch.int32, device=device)
         runs = RowSegments(table, B, N)
         kernel("gated linear attention, prompts", lambda: recurrent.gated_linear_attention(
-            ctx, yg, gw.cols[:4], zf, g, gw.head_norm, cfg.eps, runs, pos, rec, og), 0, rows * gla_row + B * state_bytes,
+            ctx, yg, gw.cols[:4], al, g, gw.head_norm, cfg.eps, runs, pos, rec, og), 0, rows * gla_row + B * state_bytes,
             "bytes: rows once; its products are not what bounds it")
     clocks = sampler.finish()
     mixers = [lc.attention is not None for lc in cfg.layers]

@@ -396,6 +396,7 @@ int b2kv_layernorm_rows(const float* y, int64_t ld_y, const int32_t* row_index, 
  *   B2KV_SEG_GLU_CLAMP  pairs (gate, up): g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1)
  *   B2KV_SEG_RELU2      max(product, 0)^2, in the storage type
  *   B2KV_SEG_SOFTCAP    limit * tanh(product / limit), fp32
+ *   B2KV_SEG_DECAY      sigmoid(product)^(1 / limit), fp32: the decays of a recurrence
  * bias is fp32 [N] (NULL: none; products without groups only).
  * x is [rows, K] with row pitch ld_x; w is [K, N] row-major with row pitch ld_w.  Group g (0 <= g < groups) reads
  * x + g * group_x and w + g * group_w and writes seg.out + g * seg.group: the heads of a per-head product.  With group_rows
@@ -412,6 +413,7 @@ int b2kv_layernorm_rows(const float* y, int64_t ld_y, const int32_t* row_index, 
 #define B2KV_SEG_GLU_CLAMP 3
 #define B2KV_SEG_RELU2 4
 #define B2KV_SEG_SOFTCAP 5
+#define B2KV_SEG_DECAY 6
 #define B2KV_MAX_SEGMENTS 3
 typedef struct b2kv_segment {
     void* out;
@@ -523,8 +525,7 @@ int b2kv_gqa_prefill(const void* q, int64_t ld_q, const void* k_cache, const voi
 /*
  * Gated linear attention: a recurrence whose state S [dim, vdim] (fp32, per sequence and head) forgets per key channel.
  * For the rows of a segment in turn, per head, with q = y[:, q_col + h * dim ...] * q_scale, k and v likewise:
- *   alpha = sigmoid(z)^(1 / tau)                     z fp32 [rows, H * dim]
- *   S <- diag(alpha) S + k v^T,  o = S^T q
+ *   S <- diag(alpha) S + k v^T,  o = S^T q           alpha in [0, 1], fp32 [rows, H * dim]
  *   out[row, h, :] = o / sqrt(mean(o^2) + eps) * norm * silu(y[row, g_col + h * vdim ...])
  * state [n_slots, H, dim, vdim] is read at the start of a segment (taken as zero where its first row's row_pos is 0) and
  * written at its end.  segments (device): rows row0 .. row0 + n - 1 belong to sequence `slot`, in order; NULL: row i is a
@@ -538,16 +539,16 @@ typedef struct b2kv_row_segment {
 } b2kv_row_segment;
 typedef struct b2kv_gla_args {
     const void* y;
-    const float* z;
+    const float* alpha;
     const float* norm;
     float* state;
     void* out;
     const b2kv_row_segment* segments;
     const int32_t* row_pos;
-    int64_t ld_y, ld_z, ld_out;
+    int64_t ld_y, ld_alpha, ld_out;
     int32_t q_col, k_col, v_col, g_col;
     int32_t H, dim, vdim, n_segments, max_n, rows, n_slots, dtype, path;
-    float q_scale, tau, eps;
+    float q_scale, eps;
 } b2kv_gla_args;
 int b2kv_gla(const b2kv_gla_args* args, int32_t* dev_status, void* stream);
 

@@ -37,7 +37,7 @@ _sz = ctypes.c_size_t
 
 _f = ctypes.c_float
 
-SEG_STORE, SEG_F32, SEG_GLU_SILU, SEG_GLU_CLAMP, SEG_RELU2, SEG_SOFTCAP = 0, 1, 2, 3, 4, 5
+SEG_STORE, SEG_F32, SEG_GLU_SILU, SEG_GLU_CLAMP, SEG_RELU2, SEG_SOFTCAP, SEG_DECAY = 0, 1, 2, 3, 4, 5, 6
 MAX_SEGMENTS = 3
 
 
@@ -60,11 +60,11 @@ class LinearArgs(ctypes.Structure):
 class GlaArgs(ctypes.Structure):
     """``b2kv_gla_args``."""
 
-    _fields_ = [("y", _vp), ("z", _vp), ("norm", _vp), ("state", _vp), ("out", _vp), ("segments", _vp), ("row_pos", _vp),
-                ("ld_y", _i64), ("ld_z", _i64), ("ld_out", _i64), ("q_col", ctypes.c_int32), ("k_col", ctypes.c_int32),
+    _fields_ = [("y", _vp), ("alpha", _vp), ("norm", _vp), ("state", _vp), ("out", _vp), ("segments", _vp), ("row_pos", _vp),
+                ("ld_y", _i64), ("ld_alpha", _i64), ("ld_out", _i64), ("q_col", ctypes.c_int32), ("k_col", ctypes.c_int32),
                 ("v_col", ctypes.c_int32), ("g_col", ctypes.c_int32), ("H", ctypes.c_int32), ("dim", ctypes.c_int32),
                 ("vdim", ctypes.c_int32), ("n_segments", ctypes.c_int32), ("max_n", ctypes.c_int32), ("rows", ctypes.c_int32),
-                ("n_slots", ctypes.c_int32), ("dtype", ctypes.c_int32), ("path", ctypes.c_int32), ("q_scale", _f), ("tau", _f),
+                ("n_slots", ctypes.c_int32), ("dtype", ctypes.c_int32), ("path", ctypes.c_int32), ("q_scale", _f),
                 ("eps", _f)]
 
 

@@ -7,7 +7,7 @@ the layer norms behind the sublayers and a 32-bit residual stream.
                    norm q over all heads, times a temperature; norm k; k, v -> cache    gqa_append
                    softmax(q k scale - slope distance) v                                gqa_decode or gqa_prefill
         gla:       [q | k | v | gate | decay rows] = x @ w_in                           linear
-                   decay logits = decay rows @ w_a2 + bias                              linear (fp32 out)
+                   decays = sigmoid(decay rows @ w_a2 + bias)^(1 / tau)                 linear (fp32 out)
                    recurrence, norm per head, gate                                      gated_linear_attention
         x += layer_norm(mixed @ w_o)                                                    linear (fp32 out), layernorm_rows
         x += layer_norm(relu(x @ w_up)^2 @ w_down)                                      linear, linear (fp32 out), layernorm_rows
@@ -28,7 +28,7 @@ from . import gqa, recurrent
 from .gqa import GqaShape
 from .kv_cache import kv_cache_create
 from .latent import PromptPlan
-from .projection import SEG_F32, SEG_RELU2, SEG_SOFTCAP, SEG_STORE, OutputSegment, linear
+from .projection import SEG_DECAY, SEG_F32, SEG_RELU2, SEG_SOFTCAP, SEG_STORE, OutputSegment, linear
 from .recurrent import GlaShape
 from .registry import register_model
 from .serving import SequenceState, ServedModel, Step, buffer1, buffer2, pad_to, sub
@@ -112,7 +112,7 @@ class LayerWeights:
     k_norm: Optional[GPUBuffer1D] = None
     slopes: Optional[GPUBuffer1D] = None
     cols: Tuple[int, ...] = ()             # gla: first columns of q, k, v, gate, decay rows
-    w_a2: Optional[GPUBuffer2D] = None     # gla: decay rows -> decay logits
+    w_a2: Optional[GPUBuffer2D] = None     # gla: decay rows -> logits of the decays
     a2_bias: Optional[GPUBuffer1D] = None
     head_norm: Optional[GPUBuffer1D] = None
     w_up: Optional[GPUBuffer2D] = None
@@ -327,13 +327,14 @@ def _attend(ctx, state: BamasunState, i: int, xs: GPUBuffer2D, step: Step) -> GP
 def _recur(ctx, state: BamasunState, i: int, xs: GPUBuffer2D, step: Step) -> GPUBuffer2D:
     g, w, T, width = state.cfg.layers[i].gla, state.weights.layers[i], step.rows, state.cfg.width
     y = state.rows(f"in{w.w_in.shape[1]}", T, w.w_in.shape[1], state.dtype)
-    z = state.rows(f"decay{w.w_a2.shape[1]}", T, w.w_a2.shape[1], torch.float32)
+    alpha = state.rows(f"decay{w.w_a2.shape[1]}", T, w.w_a2.shape[1], torch.float32)
     out = state.rows(f"mixed{w.w_o.shape[0]}", T, w.w_o.shape[0], state.dtype)
     linear(ctx, xs, w.w_in, width, [OutputSegment(y.shape[1], SEG_STORE, y)])
-    linear(ctx, sub(y, 0, T, w.cols[4]), w.w_a2, w.w_a2.shape[0], [OutputSegment(z.shape[1], SEG_F32, z)], bias=w.a2_bias)
+    linear(ctx, sub(y, 0, T, w.cols[4]), w.w_a2, w.w_a2.shape[0], [OutputSegment(alpha.shape[1], SEG_DECAY, alpha)],
+           limit=g.tau, bias=w.a2_bias)
     for segments in (step.short, step.long):
         if segments is not None:
-            recurrent.gated_linear_attention(ctx, y, w.cols[:4], z, g, w.head_norm, state.cfg.eps, segments, step.places.pos,
+            recurrent.gated_linear_attention(ctx, y, w.cols[:4], alpha, g, w.head_norm, state.cfg.eps, segments, step.places.pos,
                                              state.recurrent[i], out)
     return out
 

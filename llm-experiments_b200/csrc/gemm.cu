@@ -452,6 +452,10 @@ __device__ __forceinline__ void epilogue_rows(const SegParams& p, uint32_t t_add
         if (sg.kind == B2KV_SEG_RELU2) {
 #pragma unroll
             for (int i = 0; i < 32; ++i) acc[i] = __float_as_uint(lin::single(B2KV_SEG_RELU2, __uint_as_float(acc[i]), 0.f));
+        } else if (sg.kind == B2KV_SEG_DECAY) {
+            const float inv_tau = 1.0f / p.a.limit;
+#pragma unroll
+            for (int i = 0; i < 32; ++i) acc[i] = __float_as_uint(lin::decay(__uint_as_float(acc[i]), inv_tau));
         } else if (sg.kind == B2KV_SEG_SOFTCAP) {
 #pragma unroll
             for (int i = 0; i < 32; ++i) acc[i] = __float_as_uint(lin::single(B2KV_SEG_SOFTCAP, __uint_as_float(acc[i]), p.a.limit));

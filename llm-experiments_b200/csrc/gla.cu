@@ -53,13 +53,12 @@ __global__ void __launch_bounds__(kThreads) gla_step_kernel(const b2kv_gla_args 
     float* const part = s_q + a.dim;  // [ry_count][vdim]
     float* const state = a.state + (static_cast<int64_t>(sg.slot) * a.H + h) * a.dim * a.vdim;
     bool fresh = a.row_pos[sg.row0] == 0;
-    const float inv_tau = 1.0f / a.tau;
     for (int i = 0; i < sg.n; ++i) {
         const int64_t row = sg.row0 + i;
         const T* y = static_cast<const T*>(a.y) + row * a.ld_y;
-        const float* z = a.z + row * a.ld_z + static_cast<int64_t>(h) * a.dim;
+        const float* alpha = a.alpha + row * a.ld_alpha + static_cast<int64_t>(h) * a.dim;
         for (int d = threadIdx.x; d < a.dim; d += kThreads) {
-            s_alpha[d] = expf(log_sigmoid(z[d]) * inv_tau);
+            s_alpha[d] = alpha[d];
             s_k[d] = Elt<T>::to_float(y[a.k_col + h * a.dim + d]);
             s_q[d] = Elt<T>::to_float(y[a.q_col + h * a.dim + d]) * a.q_scale;
         }
@@ -117,8 +116,10 @@ __global__ void __launch_bounds__(kThreads) gla_step_kernel(const b2kv_gla_args 
         for (int w = 0; w < kThreads / 32; ++w) sum += red[w];
         const float scale = 1.0f / sqrtf(sum / static_cast<float>(a.vdim) + a.eps);
         T* out = static_cast<T*>(a.out) + row * a.ld_out + static_cast<int64_t>(h) * a.vdim;
-        for (int c = threadIdx.x; c < a.vdim; c += kThreads)
-            out[c] = Elt<T>::from_float(part[c] * scale * a.norm[c] * silu(Elt<T>::to_float(y[a.g_col + h * a.vdim + c])));
+        for (int c = threadIdx.x; c < a.vdim; c += kThreads) {
+            const float g = Elt<T>::to_float(y[a.g_col + h * a.vdim + c]);
+            out[c] = Elt<T>::from_float(part[c] * scale * a.norm[c] * (sizeof(T) == 4 ? silu(g) : silu_fast(g)));
+        }
         // (the next token's first barrier comes before anything of shared memory but alpha, k, q is written again, and those were
         // read before the last two)
     }
@@ -148,12 +149,12 @@ extern "C" int b2kv_gla(const b2kv_gla_args* args, int32_t* dev_status, void* st
     if (args == nullptr) return B2KV_ERR_BAD_ARG;
     const b2kv_gla_args& a = *args;
     if (elt_bytes(a.dtype) == 0) return B2KV_ERR_UNSUPPORTED;
-    if (!a.y || !a.z || !a.norm || !a.state || !a.out || !a.row_pos || a.path < 0 || a.path > 2) return B2KV_ERR_BAD_ARG;
+    if (!a.y || !a.alpha || !a.norm || !a.state || !a.out || !a.row_pos || a.path < 0 || a.path > 2) return B2KV_ERR_BAD_ARG;
     if (a.H <= 0 || a.dim <= 0 || a.vdim <= 0 || a.n_segments <= 0 || a.max_n <= 0 || a.rows <= 0 || a.n_slots <= 0) return B2KV_ERR_BAD_ARG;
     if (!a.segments && (a.n_segments > a.rows || a.n_segments > a.n_slots)) return B2KV_ERR_BAD_ARG;
     const int64_t keys = static_cast<int64_t>(a.H) * a.dim, values = static_cast<int64_t>(a.H) * a.vdim;
     if (a.q_col < 0 || a.k_col < 0 || a.v_col < 0 || a.g_col < 0 || a.ld_y < a.q_col + keys || a.ld_y < a.k_col + keys ||
-        a.ld_y < a.v_col + values || a.ld_y < a.g_col + values || a.ld_z < keys || a.ld_out < values || !(a.tau > 0.f))
+        a.ld_y < a.v_col + values || a.ld_y < a.g_col + values || a.ld_alpha < keys || a.ld_out < values)
         return B2KV_ERR_BAD_ARG;
     if (a.path == 2 || (a.path == 0 && a.dtype == B2KV_DTYPE_BF16 && a.max_n > 16)) {
         const int rc = gla_chunked(a, dev_status, stream);

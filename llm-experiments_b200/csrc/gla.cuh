@@ -12,10 +12,9 @@ int gla_chunked(const b2kv_gla_args& a, int32_t* dev_status, void* stream);
 
 namespace gla {
 
-// ln(sigmoid(z)), without cancellation on either side.
-__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
-
 __device__ __forceinline__ float silu(float g) { return g / (1.0f + expf(-g)); }
+
+__device__ __forceinline__ float silu_fast(float g) { return __fdividef(g, 1.0f + __expf(-g)); }
 
 // Segment of a CTA, and whether it lies inside the buffers.
 __device__ __forceinline__ bool segment_place(const b2kv_gla_args& a, int i, b2kv_row_segment& sg) {

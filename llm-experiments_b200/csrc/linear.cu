@@ -84,7 +84,8 @@ __global__ void __launch_bounds__(kThreads) linear_simt_kernel(const b2kv_linear
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 if (c + e >= a.N) break;
-                float v = single(sg.kind, acc[i][j + e], a.limit);
+                float v = sizeof(T) == 4 && sg.kind == B2KV_SEG_DECAY ? decay_exact(acc[i][j + e], a.limit)
+                                                                      : single(sg.kind, acc[i][j + e], a.limit);
                 if (is_f32(sg.kind)) {
                     if (a.residual != nullptr && sg.kind == B2KV_SEG_F32) v += a.residual[out_row * a.ld_residual + local + e];
                     static_cast<float*>(sg.out)[base + local + e] = v;
@@ -142,7 +143,7 @@ extern "C" int b2kv_linear(const b2kv_linear_args* args, int32_t* dev_status, vo
     int first = 0;
     for (int s = 0; s < a.n_seg; ++s) {
         const b2kv_segment& sg = a.seg[s];
-        if (!sg.out || (sg.kind == B2KV_SEG_SOFTCAP && !(a.limit > 0.f)) || sg.end <= first || sg.kind < B2KV_SEG_STORE || sg.kind > B2KV_SEG_SOFTCAP) return B2KV_ERR_BAD_ARG;
+        if (!sg.out || (sg.kind >= B2KV_SEG_SOFTCAP && !(a.limit > 0.f)) || sg.end <= first || sg.kind < B2KV_SEG_STORE || sg.kind > B2KV_SEG_DECAY) return B2KV_ERR_BAD_ARG;
         // pairs of columns never straddle a boundary (the last segment may end on an odd column if it has no pairs)
         if ((sg.end & 1) && (s + 1 < a.n_seg || lin::is_pair(sg.kind))) return B2KV_ERR_BAD_ARG;
         first = sg.end;

@@ -16,7 +16,23 @@ __device__ __forceinline__ float glu(int kind, float g, float u, float limit) {
 
 // Kinds whose columns are (gate, up) pairs; kinds whose output is fp32.
 __host__ __device__ constexpr bool is_pair(int kind) { return kind == B2KV_SEG_GLU_SILU || kind == B2KV_SEG_GLU_CLAMP; }
-__host__ __device__ constexpr bool is_f32(int kind) { return kind == B2KV_SEG_F32 || kind == B2KV_SEG_SOFTCAP; }
+__host__ __device__ constexpr bool is_f32(int kind) { return kind == B2KV_SEG_F32 || kind >= B2KV_SEG_SOFTCAP; }
+
+// sigmoid(z)^(1 / tau) through ln(sigmoid(z)) = min(z, 0) - ln(1 + u), u = exp(-|z|), which cancels on neither side.  Without
+// branches or calls: ln(1 + u) = 2 atanh(s), s = u / (2 + u) <= 1/3, as a series whose first dropped term is below 2^-26 of it.
+__device__ __forceinline__ float decay(float z, float inv_tau) {
+    const float u = __expf(-fabsf(z)), s = __fdividef(u, 2.0f + u), s2 = s * s;
+    float p = 1.0f / 15.0f;
+    p = fmaf(p, s2, 1.0f / 13.0f);
+    p = fmaf(p, s2, 1.0f / 11.0f);
+    p = fmaf(p, s2, 1.0f / 9.0f);
+    p = fmaf(p, s2, 1.0f / 7.0f);
+    p = fmaf(p, s2, 1.0f / 5.0f);
+    p = fmaf(p, s2, 1.0f / 3.0f);
+    p = fmaf(p, s2, 1.0f);
+    return __expf((fminf(z, 0.f) - 2.0f * s * p) * inv_tau);
+}
+__device__ __forceinline__ float decay_exact(float z, float tau) { return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) / tau); }
 
 // What happens to a single column before it is stored.
 __device__ __forceinline__ float single(int kind, float v, float limit) {
@@ -24,6 +40,7 @@ __device__ __forceinline__ float single(int kind, float v, float limit) {
         v = fmaxf(v, 0.f);
         return v * v;
     }
+    if (kind == B2KV_SEG_DECAY) return decay(v, 1.0f / limit);
     return kind == B2KV_SEG_SOFTCAP ? limit * tanhf(v / limit) : v;
 }
 

@@ -17,7 +17,7 @@ from typing import Optional, Sequence
 import torch
 
 from . import _native
-from ._native import SEG_F32, SEG_GLU_CLAMP, SEG_GLU_SILU, SEG_RELU2, SEG_SOFTCAP, SEG_STORE  # noqa: F401
+from ._native import SEG_DECAY, SEG_F32, SEG_GLU_CLAMP, SEG_GLU_SILU, SEG_RELU2, SEG_SOFTCAP, SEG_STORE  # noqa: F401
 from .batch import batch_op_begin, dev_status_ptr, reference_op, validate_buffer_shape_2d
 from .kv_cache import _ptr, cache_strides, dtype_code
 from .types import GPUBuffer1D, GPUBuffer2D, GPUContext, KVCache
@@ -109,7 +109,8 @@ class OutputSegment:
     """Columns of a linear layer's weight up to ``end`` (from the end of the segment before) and where their products go:
     ``SEG_STORE`` in the storage type, ``SEG_F32`` in fp32 (with the residual added), ``SEG_GLU_SILU`` / ``SEG_GLU_CLAMP``
     as gated pairs, (gate, up) in neighbouring columns, giving half as many output columns, ``SEG_RELU2`` as the square of the
-    positive part, ``SEG_SOFTCAP`` in fp32 squeezed into (-limit, limit) by a tanh.  ``out`` may be a view of some
+    positive part, ``SEG_SOFTCAP`` in fp32 squeezed into (-limit, limit) by a tanh, ``SEG_DECAY`` in fp32 as the limit-th root of a sigmoid.
+    ``out`` may be a view of some
     columns of a wider buffer; group g of a grouped product writes ``group`` elements further on per group."""
 
     end: int
@@ -142,7 +143,7 @@ def linear(ctx: GPUContext, x: GPUBuffer2D, w: GPUBuffer2D, k: int, segments: Se
                            max_group_rows=max_group_rows, n_seg=len(segments), dtype=dtype_code(x.buffer.dtype), path=path,
                            limit=limit)
     for i, s in enumerate(segments):
-        want = torch.float32 if s.kind in (SEG_F32, SEG_SOFTCAP) else x.buffer.dtype
+        want = torch.float32 if s.kind in (SEG_F32, SEG_SOFTCAP, SEG_DECAY) else x.buffer.dtype
         if s.out.buffer.dtype != want or s.out.buffer.stride(1) != 1 or s.out.shape[0] < rows:
             raise ValueError(f"linear: output of segment {i} must be {want} with at least {rows} rows of contiguous elements")
         a.seg[i] = _native.Segment(out=s.out.buffer.data_ptr(), ld=s.out.buffer.stride(0), group=s.group, end=s.end,

@@ -35,21 +35,21 @@ def gla_state_create(ctx: GPUContext, shape: GlaShape, batch_size: int) -> torch
 
 
 @reference_op("gated_linear_attention")
-def gated_linear_attention(ctx: GPUContext, y: GPUBuffer2D, cols: Tuple[int, int, int, int], z: GPUBuffer2D, shape: GlaShape,
+def gated_linear_attention(ctx: GPUContext, y: GPUBuffer2D, cols: Tuple[int, int, int, int], alpha: GPUBuffer2D, shape: GlaShape,
                            norm: GPUBuffer1D, eps: float, segments: RowSegments, pos: torch.Tensor, state: torch.Tensor,
                            out: GPUBuffer2D, path: int = 0) -> None:
     """The recurrence over the rows of ``segments``, with the heads' norm and gate behind it.  ``y`` holds queries, keys, values
-    and gates from the columns ``cols`` on, ``z`` (fp32) the decays' logits, ``pos`` every row's position.  ``path`` forces a
+    and gates from the columns ``cols`` on, ``alpha`` (fp32) the decays, ``pos`` every row's position.  ``path`` forces a
     kernel (1 token after token, 2 chunks on the tensor cores)."""
     if state.dtype != torch.float32 or tuple(state.shape[1:]) != (shape.heads, shape.dim, shape.vdim) or not state.is_contiguous():
         raise ValueError("the state does not have this layer's sizes")
-    if z.buffer.dtype != torch.float32 or out.buffer.dtype != y.buffer.dtype or norm.buffer.dtype != torch.float32:
-        raise ValueError("gated_linear_attention: z and norm are float32, out has the type of y")
+    if alpha.buffer.dtype != torch.float32 or out.buffer.dtype != y.buffer.dtype or norm.buffer.dtype != torch.float32:
+        raise ValueError("gated_linear_attention: alpha and norm are float32, out has the type of y")
     a = _native.GlaArgs(
-        y=y.buffer.data_ptr(), z=z.buffer.data_ptr(), norm=norm.buffer.data_ptr(), state=state.data_ptr(), out=out.buffer.data_ptr(),
+        y=y.buffer.data_ptr(), alpha=alpha.buffer.data_ptr(), norm=norm.buffer.data_ptr(), state=state.data_ptr(), out=out.buffer.data_ptr(),
         segments=None if segments.table is None else segments.table.data_ptr(), row_pos=pos.data_ptr(), ld_y=y.buffer.stride(0),
-        ld_z=z.buffer.stride(0), ld_out=out.buffer.stride(0), q_col=cols[0], k_col=cols[1], v_col=cols[2], g_col=cols[3],
+        ld_alpha=alpha.buffer.stride(0), ld_out=out.buffer.stride(0), q_col=cols[0], k_col=cols[1], v_col=cols[2], g_col=cols[3],
         H=shape.heads, dim=shape.dim, vdim=shape.vdim, n_segments=segments.count, max_n=segments.max_n, rows=y.shape[0],
-        n_slots=state.shape[0], dtype=dtype_code(y.buffer.dtype), path=path, q_scale=shape.dim ** -0.5, tau=shape.tau, eps=eps)
+        n_slots=state.shape[0], dtype=dtype_code(y.buffer.dtype), path=path, q_scale=shape.dim ** -0.5, eps=eps)
     stream = batch_op_begin(ctx)
     _native.check(_native.lib.b2kv_gla(ctypes.byref(a), dev_status_ptr(ctx), stream))

@@ -18,7 +18,7 @@ def wrap(pkg, t):
 
 
 class Layer:
-    """Rows of random queries, keys, values, gates and decay logits, and what the equations make of them."""
+    """Rows of random queries, keys, values, gates and decays, and what the equations make of them."""
 
     def __init__(self, pkg, heads, dim, vdim, tau, dtype, z_mean=3.0, z_std=2.0, seed=0):
         from llm_experiments_b200 import recurrent
@@ -37,7 +37,7 @@ class Layer:
     def rows(self, n):
         y = torch.randn((n, self.width), generator=self.gen, device="cuda").to(self.dtype)
         z = torch.randn((n, self.shape.heads * self.shape.dim), generator=self.gen, device="cuda") * self.z_std + self.z_mean
-        return y, z
+        return y, (torch.sigmoid(z.double()) ** (1 / self.shape.tau)).float()
 
     def states(self, slots):
         from llm_experiments_b200 import recurrent
@@ -46,7 +46,7 @@ class Layer:
         s.fill_(float("nan"))  # a run that starts at position 0 takes nothing over
         return s
 
-    def run(self, y, z, segments, pos, state, path, eps=1e-4):
+    def run(self, y, al, segments, pos, state, path, eps=1e-4):
         """``segments``: (row0, n, slot)."""
         from llm_experiments_b200 import recurrent
         from llm_experiments_b200.serving import RowSegments
@@ -55,7 +55,7 @@ class Layer:
         out = torch.full((len(y) + 1, sh.heads * sh.vdim + 8), 7.0, dtype=self.dtype, device="cuda")
         seg = RowSegments(torch.tensor(segments, dtype=torch.int32, device="cuda"), len(segments), max(n for _, n, _ in segments))
         pkg.gpu.batch_begin(self.ctx)
-        recurrent.gated_linear_attention(self.ctx, wrap(pkg, y), self.cols, wrap(pkg, z), sh,
+        recurrent.gated_linear_attention(self.ctx, wrap(pkg, y), self.cols, wrap(pkg, al), sh,
                                          pkg.gpu.GPUBuffer1D(buffer=self.norm, shape=(sh.vdim,), size=sh.vdim), eps, seg,
                                          torch.tensor(pos, dtype=torch.int32, device="cuda"), state, wrap(pkg, out[:len(y)]), path=path)
         pkg.gpu.batch_commit(self.ctx)
@@ -63,15 +63,14 @@ class Layer:
         assert (out[len(y)] == 7).all() and (out[:, sh.heads * sh.vdim:] == 7).all()
         return out[:len(y), :sh.heads * sh.vdim].double().cpu().numpy()
 
-    def want(self, y, z, state=None, eps=1e-4):
+    def want(self, y, al, state=None, eps=1e-4):
         """Output and last state of one sequence, float64."""
         sh = self.shape
         n = len(y)
-        y, z = y.double().cpu().numpy(), z.double().cpu().numpy()
+        y, alpha = y.double().cpu().numpy(), al.double().cpu().numpy().reshape(n, sh.heads, sh.dim)
         part = lambda c, d: y[:, c:c + sh.heads * d].reshape(n, sh.heads, d)  # noqa: E731
         q, k = part(self.cols[0], sh.dim) * sh.dim ** -0.5, part(self.cols[1], sh.dim)
         v, g = part(self.cols[2], sh.vdim), part(self.cols[3], sh.vdim)
-        alpha = (bo.sigmoid(z) ** (1 / sh.tau)).reshape(n, sh.heads, sh.dim)
         outs, states = [], []
         for h in range(sh.heads):
             o, s = bo.recurrence(q[:, h], k[:, h], v[:, h], alpha[:, h], None if state is None else state[h])
@@ -101,10 +100,10 @@ CASES = [(STEP, F32, 3, 5, 7), (STEP, BF, 2, 9, 33), (STEP, F32, 2, 48, 300), (S
 @pytest.mark.parametrize("n", [1, 2, 15, 16, 17, 33, 100])
 def test_whole_sequences(pkg, path, dtype, heads, dim, vdim, n):
     layer = Layer(pkg, heads, dim, vdim, 4.0, dtype, seed=n)
-    y, z = layer.rows(n)
+    y, al = layer.rows(n)
     state = layer.states(2)
-    got = layer.run(y, z, [(0, n, 1)], range(n), state, path)
-    want, last = layer.want(y, z)
+    got = layer.run(y, al, [(0, n, 1)], range(n), state, path)
+    want, last = layer.want(y, al)
     close(got, want, dtype, n)
     state_close(state[1], last)
     assert torch.isnan(state[0]).all()
@@ -115,17 +114,17 @@ def test_portions_carry_the_state(pkg, path, dtype, heads, dim, vdim):
     """Any cut gives the outputs of the whole, with two sequences in unequal portions per call and the rows of a call in any
     order; both kernels take turns when the choice is left open."""
     layer = Layer(pkg, heads, dim, vdim, 8.0, dtype, seed=3)
-    (ya, za), (yb, zb) = layer.rows(143), layer.rows(90)
-    wa, sa = layer.want(ya, za)
-    wb, sb = layer.want(yb, zb)
+    (ya, ala), (yb, alb) = layer.rows(143), layer.rows(90)
+    wa, sa = layer.want(ya, ala)
+    wb, sb = layer.want(yb, alb)
     state = layer.states(3)
     at = [0, 0]
     for na, nb in [(2, 40), (30, 1), (1, 2), (64, 16), (17, 31), (29, 0)]:
         ra, rb = slice(at[0], at[0] + na), slice(at[1], at[1] + nb)
-        y, z = torch.cat([yb[rb], ya[ra]]), torch.cat([zb[rb], za[ra]])
+        y, al = torch.cat([yb[rb], ya[ra]]), torch.cat([alb[rb], ala[ra]])
         segs = ([(0, nb, 2)] if nb else []) + [(nb, na, 0)]
         pos = list(range(rb.start, rb.stop)) + list(range(ra.start, ra.stop))
-        got = layer.run(y, z, segs, pos, state, path)
+        got = layer.run(y, al, segs, pos, state, path)
         if nb:
             close(got[:nb], wb[rb], dtype, (na, nb))
         close(got[nb:], wa[ra], dtype, (na, nb))
@@ -140,10 +139,10 @@ def test_portions_carry_the_state(pkg, path, dtype, heads, dim, vdim):
 def test_strong_and_vanishing_decays(pkg, path, dtype, z_mean, z_std, tau):
     """Channels that forget everything at once, that forget nothing, and both in turn: nothing overflows and nothing is lost."""
     layer = Layer(pkg, 2, 40, 48, tau, dtype, z_mean, z_std, seed=5)
-    y, z = layer.rows(75)
+    y, al = layer.rows(75)
     state = layer.states(1)
-    got = layer.run(y, z, [(0, 75, 0)], range(75), state, path)
-    want, last = layer.want(y, z)
+    got = layer.run(y, al, [(0, 75, 0)], range(75), state, path)
+    want, last = layer.want(y, al)
     close(got, want, dtype)
     state_close(state[0], last)
 
@@ -152,14 +151,14 @@ def test_strong_and_vanishing_decays(pkg, path, dtype, z_mean, z_std, tau):
 def test_a_far_token_is_remembered_for_hundreds_of_tokens(pkg, path, dtype):
     """Without decay the value written at token 3 is read back by the only query that matches its key, 500 tokens later."""
     layer = Layer(pkg, 1, 16, 32, 1.0, dtype, z_mean=80.0, z_std=0.0, seed=7)
-    y, z = layer.rows(520)
+    y, al = layer.rows(520)
     c = layer.cols
     y[:, c[0]:c[0] + 16], y[:, c[1]:c[1] + 16] = 0, 0
     y[:, c[1] + 1] = 1.0         # every key is unit vector 1 ...
     y[3, c[1]:c[1] + 16] = 0
     y[3, c[1] + 9] = 1.0         # ... but token 3's is unit vector 9
     y[503, c[0] + 9] = 4.0
-    got = layer.run(y, z, [(0, 520, 0)], range(520), layer.states(1), path)
+    got = layer.run(y, al, [(0, 520, 0)], range(520), layer.states(1), path)
     v, g = (y[r, k:k + 32].double().cpu().numpy() for r, k in ((3, c[2]), (503, c[3])))
     close(got[503], bo.rms_norm(v, layer.norm.double().cpu().numpy(), 1e-4) * g * bo.sigmoid(g), dtype)
     assert np.abs(got[502]).max() == 0  # (a query of zeros)
@@ -173,24 +172,24 @@ def test_a_decode_step_takes_one_row_per_sequence(pkg):
     layer = Layer(pkg, 4, 64, 96, 16.0, BF, seed=9)
     state = torch.randn((3, 4, 64, 96), generator=layer.gen, device="cuda")
     before = state.double().cpu().numpy()
-    y, z = layer.rows(3)
+    y, al = layer.rows(3)
     out = torch.empty((3, 4 * 96), dtype=BF, device="cuda")
     pos = torch.tensor([12, 0, 1], dtype=torch.int32, device="cuda")
     pkg.gpu.batch_begin(layer.ctx)
-    recurrent.gated_linear_attention(layer.ctx, wrap(pkg, y), layer.cols, wrap(pkg, z), layer.shape,
+    recurrent.gated_linear_attention(layer.ctx, wrap(pkg, y), layer.cols, wrap(pkg, al), layer.shape,
                                      pkg.gpu.GPUBuffer1D(buffer=layer.norm, shape=(96,), size=96), 1e-4, RowSegments(None, 3, 1), pos, state,
                                      wrap(pkg, out))
     pkg.gpu.batch_commit(layer.ctx)
     for i in range(3):
-        want, last = layer.want(y[i:i + 1], z[i:i + 1], None if i == 1 else before[i])
+        want, last = layer.want(y[i:i + 1], al[i:i + 1], None if i == 1 else before[i])
         close(out[i:i + 1].double().cpu().numpy(), want, BF, i)
         state_close(state[i], last)
 
 
 def test_segments_outside_the_buffers_are_refused(pkg):
     layer = Layer(pkg, 2, 16, 16, 2.0, BF)
-    y, z = layer.rows(20)
+    y, al = layer.rows(20)
     for path in (STEP, CHUNK):
         for seg in ((0, 21, 0), (5, 16, 0), (0, 20, 1), (-1, 4, 0)):
             with pytest.raises(RuntimeError, match="position"):
-                layer.run(y, z, [seg], range(20), layer.states(1), path)
+                layer.run(y, al, [seg], range(20), layer.states(1), path)
