@@ -405,7 +405,9 @@ int b2kv_layernorm_rows(const float* y, int64_t ld_y, const int32_t* row_index, 
  * Offsets and pitches are in elements.  Segment boundaries are even.  The product runs on the tensor cores for bf16 when
  * pitches, offsets and boundaries allow it (multiples of 8 elements; boundaries multiples of 32): at most 128 rows per
  * group stream the weights once, more go to the tiled kernel; everything else, and fp32, runs on a CUDA-core kernel.
- * path: 0 = choose, 1 = CUDA cores, 2 = weight streaming, 3 = tiled (refused when the shape is not one it takes).
+ * A bf16 product of one segment with at most 32 input features runs on a CUDA-core kernel of its own.
+ * path: 0 = choose, 1 = CUDA cores, 2 = weight streaming, 3 = tiled, 4 = few input features (refused when the shape is not one
+ * it takes).
  */
 #define B2KV_SEG_STORE 0
 #define B2KV_SEG_F32 1

@@ -184,8 +184,7 @@ def prepare_weights(ctx: GPUContext, cfg: BamasunConfig, tensors: Dict[str, torc
                 cols.append(pad_to(cols[-1] + n, 8))
             w_in = stack([(c, p + "mix." + name, n, width)
                           for c, name, n in zip(cols, ("q", "k", "v", "g", "a1"), (nk, nk, nv, nv, rank))], width)
-            # (the last part is as wide as what is left of the padded columns: its zero columns meet zero rows)
-            w_a2 = stack([(0, p + "mix.a2", nk, rank)], w_in.shape[1] - cols[4])
+            w_a2 = stack([(0, p + "mix.a2", nk, rank)], pad_to(rank, 8))
             lw = LayerWeights(w_in=w_in, w_o=stack([(0, p + "mix.o", width, nv)], pad_to(nv, 16)), norm1=norm(p + "norm1"),
                               cols=tuple(cols), w_a2=w_a2, a2_bias=vector(p + "mix.a2.b", nk, w_a2.shape[1]),
                               head_norm=vector(p + "mix.norm", g.vdim))

@@ -21,41 +21,68 @@ __device__ __forceinline__ void narrow_store(__nv_bfloat16* p, const float (&f)[
     *reinterpret_cast<uint4*>(p) = *reinterpret_cast<uint4*>(h);
 }
 
-// Sum of squares of src[0, n) seen by this thread; n and src in whole 16-byte pieces when kVec.
-template <typename T, bool kVec>
-__device__ __forceinline__ float squares(const T* src, int n) {
-    float sum = 0.f;
-    if (kVec) {
-        constexpr int kC = Elt<T>::kPerChunk;
-        for (int i = threadIdx.x; i < n / kC; i += kAppendThreads) {
-            float f[kC];
-            Elt<T>::widen(reinterpret_cast<const uint4*>(src)[i], f);
-#pragma unroll
-            for (int e = 0; e < kC; ++e) sum = fmaf(f[e], f[e], sum);
-        }
-    } else {
-        for (int i = threadIdx.x; i < n; i += kAppendThreads) sum = fmaf(Elt<T>::to_float(src[i]), Elt<T>::to_float(src[i]), sum);
+// This thread's share of a row of n elements: 16-byte pieces when kVec (n a whole number of them), the first kKeep of which
+// stay in registers.
+template <typename T, bool kVec, int kKeep>
+struct Row {
+    static constexpr int kC = Elt<T>::kPerChunk;
+    uint4 keep[kKeep];
+    __device__ __forceinline__ uint4 piece(const T* src, int j) const {
+        return reinterpret_cast<const uint4*>(src)[threadIdx.x + j * kAppendThreads];
     }
-    return sum;
-}
-
-// dst = src * factor * w (w NULL: src * factor); dst may be src.
-template <typename T, bool kVec>
-__device__ __forceinline__ void scaled(T* dst, const T* src, const float* w, float factor, int n) {
-    if (kVec) {
-        constexpr int kC = Elt<T>::kPerChunk;
-        for (int i = threadIdx.x; i < n / kC; i += kAppendThreads) {
-            float f[kC];
-            Elt<T>::widen(reinterpret_cast<const uint4*>(src)[i], f);
+    __device__ __forceinline__ void load(const T* src, int n) {
+        if (!kVec) return;
 #pragma unroll
-            for (int e = 0; e < kC; ++e) f[e] *= w != nullptr ? factor * w[i * kC + e] : factor;
-            narrow_store(dst + i * kC, f);
-        }
-    } else {
-        for (int i = threadIdx.x; i < n; i += kAppendThreads)
-            dst[i] = Elt<T>::from_float(Elt<T>::to_float(src[i]) * (w != nullptr ? factor * w[i] : factor));
+        for (int j = 0; j < kKeep; ++j)
+            if (static_cast<int>(threadIdx.x) + j * kAppendThreads < n / kC) keep[j] = piece(src, j);
     }
-}
+    // fn(piece, index of its first element)
+    template <typename F>
+    __device__ __forceinline__ void each(const T* src, int n, F&& fn) const {
+#pragma unroll
+        for (int j = 0; j < kKeep; ++j)
+            if (static_cast<int>(threadIdx.x) + j * kAppendThreads < n / kC) fn(keep[j], (threadIdx.x + j * kAppendThreads) * kC);
+        for (int j = kKeep; static_cast<int>(threadIdx.x) + j * kAppendThreads < n / kC; ++j)
+            fn(piece(src, j), (threadIdx.x + j * kAppendThreads) * kC);
+    }
+    __device__ __forceinline__ float squares(const T* src, int n) const {
+        float sum = 0.f;
+        if (kVec) {
+            each(src, n, [&](const uint4& p, int) {
+                float f[kC];
+                Elt<T>::widen(p, f);
+#pragma unroll
+                for (int e = 0; e < kC; ++e) sum = fmaf(f[e], f[e], sum);
+            });
+        } else {
+            for (int i = threadIdx.x; i < n; i += kAppendThreads) sum = fmaf(Elt<T>::to_float(src[i]), Elt<T>::to_float(src[i]), sum);
+        }
+        return sum;
+    }
+    // dst = src * factor * w (w NULL: src * factor); dst may be src.
+    __device__ __forceinline__ void scaled(T* dst, const T* src, const float* w, float factor, int n) const {
+        if (kVec) {
+            each(src, n, [&](const uint4& p, int at) {
+                float f[kC];
+                Elt<T>::widen(p, f);
+                if (w != nullptr) {
+#pragma unroll
+                    for (int e = 0; e < kC; e += 4) {
+                        const float4 wv = *reinterpret_cast<const float4*>(w + at + e);
+                        f[e] *= factor * wv.x, f[e + 1] *= factor * wv.y, f[e + 2] *= factor * wv.z, f[e + 3] *= factor * wv.w;
+                    }
+                } else {
+#pragma unroll
+                    for (int e = 0; e < kC; ++e) f[e] *= factor;
+                }
+                narrow_store(dst + at, f);
+            });
+        } else {
+            for (int i = threadIdx.x; i < n; i += kAppendThreads)
+                dst[i] = Elt<T>::from_float(Elt<T>::to_float(src[i]) * (w != nullptr ? factor * w[i] : factor));
+        }
+    }
+};
 
 struct AppendArgs {
     const float *q_norm, *k_norm;
@@ -79,10 +106,15 @@ __global__ void __launch_bounds__(kAppendThreads) gqa_append_kernel(T* y, T* k_c
     }
     const int nq = a.H * a.dim, nk = a.G * a.dim, nv = a.G * a.vdim;
     T* q = y + static_cast<int64_t>(blockIdx.x) * a.ld_y;
-    T *k = q + nq, *v = k + nk;
+    const T *k = q + nq, *v = k + nk;
     const bool own = k_cache != nullptr;
-    float sq = a.q_norm != nullptr ? squares<T, kVec>(q, nq) : 0.f;
-    float sk = own && a.k_norm != nullptr ? squares<T, kVec>(k, nk) : 0.f;
+    // the first pieces of q, k and v stay in registers between the two passes, all loads on their way together
+    Row<T, kVec, 2> rq;
+    Row<T, kVec, 1> rk, rv;
+    rq.load(q, nq);
+    if (own) rk.load(k, nk), rv.load(v, nv);
+    float sq = a.q_norm != nullptr ? rq.squares(q, nq) : 0.f;
+    float sk = own && a.k_norm != nullptr ? rk.squares(k, nk) : 0.f;
 #pragma unroll
     for (int off = 16; off > 0; off >>= 1) {
         sq += __shfl_xor_sync(0xffffffffu, sq, off);
@@ -95,18 +127,12 @@ __global__ void __launch_bounds__(kAppendThreads) gqa_append_kernel(T* y, T* k_c
     for (int i = 0; i < kAppendThreads / 32; ++i) sq += part[0][i], sk += part[1][i];
     float fq = a.q_norm != nullptr ? 1.0f / sqrtf(sq / static_cast<float>(nq) + a.eps) : 1.f;
     if (a.temp_every > 0) fq *= 1.0f + a.temp_coef * logf(static_cast<float>((pos + 1) / a.temp_every) + 1.0f);
-    if (a.q_norm != nullptr || a.temp_every > 0) scaled<T, kVec>(q, q, a.q_norm, fq, nq);
+    if (a.q_norm != nullptr || a.temp_every > 0) rq.scaled(q, q, a.q_norm, fq, nq);
     if (!own) return;
     const int64_t place = static_cast<int64_t>(slot) * a.T_max + pos;
     const float fk = a.k_norm != nullptr ? 1.0f / sqrtf(sk / static_cast<float>(nk) + a.eps) : 1.f;
-    scaled<T, kVec>(k_cache + place * nk, k, a.k_norm, fk, nk);
-    T* dst = v_cache + place * nv;
-    if (kVec) {
-        for (int i = threadIdx.x; i < nv / Elt<T>::kPerChunk; i += kAppendThreads)
-            reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(v)[i];
-    } else {
-        for (int i = threadIdx.x; i < nv; i += kAppendThreads) dst[i] = v[i];
-    }
+    rk.scaled(k_cache + place * nk, k, a.k_norm, fk, nk);
+    rv.scaled(v_cache + place * nv, v, nullptr, 1.f, nv);
 }
 
 // One CTA per (head, query row); its warps take the visible tokens in turn, each with an online softmax of its own, and are
@@ -198,7 +224,7 @@ int launch_simt(const GqaDecodeArgs& a, void* stream) {
 template <typename T>
 int launch_append(T* y, T* k, T* v, const AppendArgs& a, int rows, void* stream) {
     constexpr int per = 16 / static_cast<int>(sizeof(T));
-    const bool vec = aligned16(y) && aligned16(k) && aligned16(v) && a.ld_y % per == 0 && (a.H * a.dim) % per == 0 &&
+    const bool vec = aligned16(y) && aligned16(a.q_norm) && aligned16(a.k_norm) && aligned16(k) && aligned16(v) && a.ld_y % per == 0 && (a.H * a.dim) % per == 0 &&
                      (a.G * a.dim) % per == 0 && (a.G * a.vdim) % per == 0;
     OverlapLaunch launch(rows, kAppendThreads, 0, stream);
     B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, vec ? gqa_append_kernel<T, true> : gqa_append_kernel<T, false>, y, k, v, a));

@@ -282,13 +282,16 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
             const int lo = p.window > 0 ? hi - p.window + 1 : -1;
             const float2 c2 = make_float2(c, c);
             if (kBias) {
-                // element e is hi - e tokens behind the query
-                const float base = -slope * static_cast<float>(hi);
-                const float2 slope2 = make_float2(slope, slope), base2 = make_float2(base, base);
+                // element e is hi - e tokens behind the query; four pairs of biases go along, eight elements at a step
+                float2 b[4];
+#pragma unroll
+                for (int a = 0; a < 4; ++a) b[a] = make_float2(slope * static_cast<float>(2 * a - hi), slope * static_cast<float>(2 * a + 1 - hi));
+                const float2 step = make_float2(8.f * slope, 8.f * slope);
 #pragma unroll
                 for (int e = 0; e < 128; e += 2) {
-                    const float2 b = __ffma2_rn(make_float2(static_cast<float>(e), static_cast<float>(e + 1)), slope2, base2);
-                    const float2 z = __ffma2_rn(make_float2(__uint_as_float(r[e]), __uint_as_float(r[e + 1])), c2, b);
+                    float2& be = b[(e >> 1) & 3];
+                    const float2 z = __ffma2_rn(make_float2(__uint_as_float(r[e]), __uint_as_float(r[e + 1])), c2, be);
+                    be = __fadd2_rn(be, step);
                     r[e] = __float_as_uint(z.x);
                     r[e + 1] = __float_as_uint(z.y);
                 }

@@ -1,5 +1,5 @@
 // b2kv_linear: argument checks, the choice of the kernel, and the CUDA-core kernel for fp32 and for shapes that the
-// tensor-core kernels do not take (64 x 64 output tiles, 16 input features per step, 4 x 4 outputs per thread, fp32
+// tensor-core kernels do not take, and the one for few input features (64 x 64 output tiles, 16 input features per step, 4 x 4 outputs per thread, fp32
 // accumulation).
 #include "linear.cuh"
 
@@ -110,6 +110,76 @@ static int launch_simt(const b2kv_linear_args& a, void* stream) {
     return B2KV_OK;
 }
 
+// Products with few input features (a low-rank bottleneck): what they cost is the outputs, so there is nothing for the tensor
+// cores to win.  A thread keeps two columns of w in registers and goes through a tile of rows, whose few elements lie in shared
+// memory; neighbouring threads store neighbouring columns.
+constexpr int kThinK = 32, kThinThreads = 128, kThinRows = 64;
+
+template <int kK>
+__global__ void __launch_bounds__(kThinThreads) linear_thin_kernel(const __grid_constant__ b2kv_linear_args a, int row_tile) {
+    __shared__ float4 xs[kThinRows][kK / 4];
+    const int c = (blockIdx.x * kThinThreads + threadIdx.x) * 2;
+    const bool live = c < a.N;
+    const __nv_bfloat16* const w = static_cast<const __nv_bfloat16*>(a.w);
+    float2 wr[kK], bias = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int k = 0; k < kK; ++k) {
+        wr[k] = make_float2(0.f, 0.f);
+        if (live && k < a.K) wr[k] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(w + k * a.ld_w + c));
+    }
+    if (live && a.bias != nullptr) bias = make_float2(a.bias[c], a.bias[c + 1]);
+    grid_launch_dependents();
+    if (threadIdx.x == 0) grid_dependency_wait();
+    __syncthreads();
+    const int row0 = blockIdx.y * row_tile, n = min(row_tile, a.rows - row0);
+    const __nv_bfloat16* const x = static_cast<const __nv_bfloat16*>(a.x) + row0 * a.ld_x;
+    for (int i = threadIdx.x; i < n * kK; i += kThinThreads) {
+        const int r = i / kK, k = i % kK;
+        reinterpret_cast<float*>(xs[r])[k] = k < a.K ? __bfloat162float(x[r * a.ld_x + k]) : 0.f;
+    }
+    __syncthreads();
+    if (!live) return;
+    const b2kv_segment& sg = a.seg[0];
+    for (int r = 0; r < n; ++r) {
+        float2 v = bias;
+#pragma unroll
+        for (int k = 0; k < kK; k += 4) {
+            const float4 xv = xs[r][k / 4];
+            v = __ffma2_rn(make_float2(xv.x, xv.x), wr[k], v);
+            v = __ffma2_rn(make_float2(xv.y, xv.y), wr[k + 1], v);
+            v = __ffma2_rn(make_float2(xv.z, xv.z), wr[k + 2], v);
+            v = __ffma2_rn(make_float2(xv.w, xv.w), wr[k + 3], v);
+        }
+        v.x = single(sg.kind, v.x, a.limit);
+        v.y = single(sg.kind, v.y, a.limit);
+        const int64_t row = row0 + r;
+        if (is_f32(sg.kind)) {
+            if (a.residual != nullptr && sg.kind == B2KV_SEG_F32) {
+                const float2 add = *reinterpret_cast<const float2*>(a.residual + row * a.ld_residual + c);
+                v.x += add.x, v.y += add.y;
+            }
+            *reinterpret_cast<float2*>(static_cast<float*>(sg.out) + row * sg.ld + c) = v;
+        } else {
+            *reinterpret_cast<__nv_bfloat162*>(static_cast<__nv_bfloat16*>(sg.out) + row * sg.ld + c) = __floats2bfloat162_rn(v.x, v.y);
+        }
+    }
+}
+
+static int launch_thin(const b2kv_linear_args& a, void* stream) {
+    const b2kv_segment& sg = a.seg[0];
+    if (a.dtype != B2KV_DTYPE_BF16 || a.K > kThinK || a.N % 2 || a.groups > 1 || a.group_rows || a.n_seg > 1 || is_pair(sg.kind))
+        return B2KV_ERR_UNSUPPORTED;
+    if (!aligned16(a.w) || !aligned16(sg.out) || a.ld_w % 2 || sg.ld % 2 || (a.residual && (!aligned16(a.residual) || a.ld_residual % 2)))
+        return B2KV_ERR_UNSUPPORTED;
+    // few rows: enough CTAs to be quick; many: the columns of w are loaded once per tile of rows
+    const int row_tile = a.rows > 1024 ? kThinRows : 8;
+    const dim3 grid((a.N / 2 + kThinThreads - 1) / kThinThreads, (a.rows + row_tile - 1) / row_tile);
+    if (grid.y > 65535u) return B2KV_ERR_UNSUPPORTED;
+    OverlapLaunch launch(grid, kThinThreads, 0, stream);
+    B2KV_CUDA_TRY(cudaLaunchKernelEx(&launch.cfg, a.K <= 16 ? linear_thin_kernel<16> : linear_thin_kernel<32>, a, row_tile));
+    return B2KV_OK;
+}
+
 // A per-head product of many rows: the weight-streaming kernel on 128 rows at a time (the heads' matrices are small and
 // stay in L2).
 static int rows_in_slices(const b2kv_linear_args& all, int32_t* dev_status, void* stream) {
@@ -136,7 +206,7 @@ extern "C" int b2kv_linear(const b2kv_linear_args* args, int32_t* dev_status, vo
     if (args == nullptr) return B2KV_ERR_BAD_ARG;
     const b2kv_linear_args& a = *args;
     if (elt_bytes(a.dtype) == 0) return B2KV_ERR_UNSUPPORTED;
-    if (!a.x || !a.w || a.rows <= 0 || a.K <= 0 || a.N <= 0 || a.groups <= 0 || a.path < 0 || a.path > 3) return B2KV_ERR_BAD_ARG;
+    if (!a.x || !a.w || a.rows <= 0 || a.K <= 0 || a.N <= 0 || a.groups <= 0 || a.path < 0 || a.path > 4) return B2KV_ERR_BAD_ARG;
     if (a.n_seg < 1 || a.n_seg > B2KV_MAX_SEGMENTS || a.seg[a.n_seg - 1].end != a.N) return B2KV_ERR_BAD_ARG;
     if (a.bias && a.groups > 1) return B2KV_ERR_BAD_ARG;
     if (a.group_rows && (a.max_group_rows <= 0 || a.max_group_rows > a.rows)) return B2KV_ERR_BAD_ARG;
@@ -150,8 +220,10 @@ extern "C" int b2kv_linear(const b2kv_linear_args* args, int32_t* dev_status, vo
     }
     if (a.path == 2) return linear_rows_tc(a, dev_status, stream);
     if (a.path == 3) return linear_tiled_tc(a, dev_status, stream);
+    if (a.path == 4) return lin::launch_thin(a, stream);
     if (a.path == 0 && a.dtype == B2KV_DTYPE_BF16) {
-        int rc;
+        int rc = lin::launch_thin(a, stream);
+        if (rc != B2KV_ERR_UNSUPPORTED) return rc;
         if ((a.group_rows ? a.max_group_rows : a.rows) <= 128) {
             rc = linear_rows_tc(a, dev_status, stream);
         } else if (a.groups > 1 && a.group_rows == nullptr) {

@@ -130,7 +130,7 @@ def linear(ctx: GPUContext, x: GPUBuffer2D, w: GPUBuffer2D, k: int, segments: Se
     ``groups`` > 1, group g reads ``x`` from element ``g * group_x`` on and ``w`` from ``g * group_w`` on (the heads of a
     per-head product), or, with ``group_rows`` (int32 ``[groups + 1]`` on the device), rows ``group_rows[g] ..
     group_rows[g + 1] - 1`` of ``x`` (the experts of a mixture; at most ``max_group_rows`` rows each).  ``path`` forces a
-    kernel (1 CUDA cores, 2 weight streaming, 3 tiled)."""
+    kernel (1 CUDA cores, 2 weight streaming, 3 tiled, 4 few input features)."""
     rows, n = x.shape[0], segments[-1].end
     if rows <= 0 or k <= 0 or n <= 0:
         raise ValueError(f"linear: Invalid dimensions x=({rows}, {k}), w=({k}, {n})")

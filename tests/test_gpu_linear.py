@@ -8,7 +8,7 @@ from tests.kv_util import make_ctx
 
 pytestmark = pytest.mark.gpu
 
-SIMT, ROWS, TILED = 1, 2, 3
+SIMT, ROWS, TILED, THIN = 1, 2, 3, 4
 
 
 def glu(kind, g, u, limit, proj):
@@ -143,3 +143,50 @@ def test_rows_grouped_by_expert(pkg, path, dtype, counts, K, n, glu_kind):
         prod = x[offs[e]:offs[e + 1]].double() @ w[e * K:(e + 1) * K].double()
         close(out[offs[e]:offs[e + 1]], glu(kind, prod[:, 0::2], prod[:, 1::2], 0, proj) if glu_kind else prod, dtype)
     assert (out[R] == 7).all()
+
+
+def activated(kind, z, limit, proj):
+    if kind == proj.SEG_RELU2:
+        return z.clamp(min=0) ** 2
+    if kind == proj.SEG_SOFTCAP:
+        return limit * torch.tanh(z / limit)
+    return torch.exp(torch.nn.functional.logsigmoid(z) / limit) if kind == proj.SEG_DECAY else z
+
+
+@pytest.mark.parametrize("kind", ["SEG_STORE", "SEG_F32", "SEG_RELU2", "SEG_SOFTCAP", "SEG_DECAY"])
+@pytest.mark.parametrize("path,dtype,rows,K,n", [
+    (SIMT, torch.float32, 9, 40, 21), (SIMT, torch.bfloat16, 70, 100, 33), (ROWS, torch.bfloat16, 3, 72, 40), (ROWS, torch.bfloat16, 100, 2048, 104),
+    (ROWS, torch.bfloat16, 64, 4096, 128), (TILED, torch.bfloat16, 200, 256, 208), (TILED, torch.bfloat16, 700, 136, 72),
+    (THIN, torch.bfloat16, 5, 16, 34), (THIN, torch.bfloat16, 1100, 24, 300), (THIN, torch.bfloat16, 65, 32, 256), (0, torch.bfloat16, 40, 8, 64)])
+def test_bias_and_single_column_forms(pkg, kind, path, dtype, rows, K, n):
+    """A bias added ahead of the square of the positive part, a soft cap, the root of a sigmoid, or nothing."""
+    from llm_experiments_b200 import projection as proj
+
+    ctx, kind = make_ctx(pkg), getattr(proj, kind)
+    pad = (n + 7) // 8 * 8
+    x, w = rnd((rows, K), dtype, 20), rnd((K, pad), dtype, 21, 2 * K ** -0.5)
+    bias = rnd((n,), torch.float32, 22, 2.0)
+    fp32 = kind in (proj.SEG_F32, proj.SEG_SOFTCAP, proj.SEG_DECAY)
+    out = torch.full((rows + 1, pad), 7.0, dtype=torch.float32 if fp32 else dtype, device="cuda")
+    run(pkg, ctx, wrap(pkg, x), wrap(pkg, w), K, [proj.OutputSegment(n, kind, wrap(pkg, out))], limit=2.5, path=path,
+        bias=pkg.gpu.GPUBuffer1D(buffer=bias, shape=(n,), size=n))
+    want = activated(kind, x.double() @ w.double()[:, :n] + bias.double(), 2.5, proj)
+    close(out[:rows, :n], want, torch.float32 if fp32 else dtype)
+    assert (out[rows] == 7).all() and (out[:, n:] == 7).all()
+
+
+@pytest.mark.parametrize("path,rows", [(SIMT, 6), (ROWS, 6), (TILED, 160), (THIN, 6)])
+def test_decays_close_to_one_keep_what_they_take_away(pkg, path, rows):
+    """For large logits the decay is one minus something tiny; far below zero it is a tiny number of its own."""
+    from llm_experiments_b200 import projection as proj
+
+    ctx = make_ctx(pkg)
+    z = torch.tensor([-120.0, -60.0, -20.0, -3.0, -0.5, 0.0, 0.5, 3.0, 8.0, 12.0, 14.0, 20.0, 40.0, 90.0, 1.0, -1.0], device="cuda")
+    x, w = torch.zeros((rows, 16), dtype=torch.bfloat16, device="cuda"), torch.zeros((16, 16), dtype=torch.bfloat16, device="cuda")
+    out = torch.empty((rows, 16), device="cuda")
+    for tau in (1.0, 16.0):
+        run(pkg, ctx, wrap(pkg, x), wrap(pkg, w), 16, [proj.OutputSegment(16, proj.SEG_DECAY, wrap(pkg, out))], limit=tau, path=path,
+            bias=pkg.gpu.GPUBuffer1D(buffer=z, shape=(16,), size=16))
+        want = torch.exp(torch.nn.functional.logsigmoid(z.double()) / tau)
+        torch.testing.assert_close(out[rows - 1].double(), want, rtol=2e-6 if tau == 16 else 2e-5, atol=1e-12)
+        torch.testing.assert_close(1 - out[0].double(), 1 - want, rtol=2e-3, atol=3e-7)
