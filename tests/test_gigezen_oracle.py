@@ -129,7 +129,7 @@ def test_prompt_plan_counts_blocks_and_visible_rows(pkg):
 def test_entry_points_check_their_arguments_before_any_launch(pkg):
     native = pkg._native
     lib, A = native.lib, 0x1000
-    assert lib.b2kv_embed_rows(None, A, A, 1, 8, 8, 0, None, None) == -1
+    assert lib.b2kv_embed_rows(None, A, A, None, 1.0, 1, 8, 8, 0, None, None) == -1
     assert lib.b2kv_rmsnorm(A, 8, None, A, 1.0, A, 4, 1, 8, 1e-6, 0, None) == -1  # output pitch below the row
     args = native.LinearArgs(x=A, w=A, ld_x=8, ld_w=8, rows=1, K=8, N=8, groups=1, n_seg=1, dtype=1)
     args.seg[0] = native.Segment(out=A, ld=8, end=6, kind=0)
