@@ -533,8 +533,9 @@ int b2kv_gqa_prefill(const void* q, int64_t ld_q, const void* k_cache, const voi
  * written at its end.  segments (device): rows row0 .. row0 + n - 1 belong to sequence `slot`, in order; NULL: row i is a
  * segment of its own, of sequence i.  max_n bounds the segments' lengths.  Everything is computed in 32-bit; path 2 (segments
  * of a prompt; bf16, dim a multiple of 8 up to 128, vdim a multiple of 8 up to 256) takes sixteen tokens at a time through the tensor
- * cores with operands split into two bf16 halves and the state in fp32 registers, path 1 takes token after token on CUDA
- * cores for any sizes and both types; 0 = choose.
+ * cores with operands split into two bf16 halves and the state in fp32 registers, and wants a workspace (128-byte aligned) of
+ * b2kv_gla_workspace_bytes bytes; path 1 takes token after token on CUDA cores for any sizes and both types; 0 = choose (path 2
+ * for segments of more than 16 tokens where the sizes have that form).
  */
 typedef struct b2kv_row_segment {
     int32_t row0, n, slot;
@@ -547,11 +548,14 @@ typedef struct b2kv_gla_args {
     void* out;
     const b2kv_row_segment* segments;
     const int32_t* row_pos;
+    void* workspace;
+    size_t workspace_bytes;
     int64_t ld_y, ld_alpha, ld_out;
     int32_t q_col, k_col, v_col, g_col;
     int32_t H, dim, vdim, n_segments, max_n, rows, n_slots, dtype, path;
     float q_scale, eps;
 } b2kv_gla_args;
+size_t b2kv_gla_workspace_bytes(int H, int dim, int vdim, int n_segments, int max_n, int dtype, int path);
 int b2kv_gla(const b2kv_gla_args* args, int32_t* dev_status, void* stream);
 
 /*

@@ -60,7 +60,8 @@ class LinearArgs(ctypes.Structure):
 class GlaArgs(ctypes.Structure):
     """``b2kv_gla_args``."""
 
-    _fields_ = [("y", _vp), ("alpha", _vp), ("norm", _vp), ("state", _vp), ("out", _vp), ("segments", _vp), ("row_pos", _vp),
+    _fields_ = [("y", _vp), ("alpha", _vp), ("norm", _vp), ("state", _vp), ("out", _vp), ("segments", _vp), ("row_pos", _vp), ("workspace", _vp),
+                ("workspace_bytes", _sz),
                 ("ld_y", _i64), ("ld_alpha", _i64), ("ld_out", _i64), ("q_col", ctypes.c_int32), ("k_col", ctypes.c_int32),
                 ("v_col", ctypes.c_int32), ("g_col", ctypes.c_int32), ("H", ctypes.c_int32), ("dim", ctypes.c_int32),
                 ("vdim", ctypes.c_int32), ("n_segments", ctypes.c_int32), ("max_n", ctypes.c_int32), ("rows", ctypes.c_int32),
@@ -124,6 +125,7 @@ SIGNATURES = {
                              _vp, _vp]),
     "b2kv_gqa_prefill_supported": (_i, [_i, _i, _i]),
     "b2kv_gqa_prefill": (_i, [_vp, _i64, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp]),
+    "b2kv_gla_workspace_bytes": (_sz, [_i, _i, _i, _i, _i, _i, _i]),
     "b2kv_gla": (_i, [ctypes.POINTER(GlaArgs), _vp, _vp]),
     "b2kv_route": (_i, [_vp, _i64, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp]),
     "b2kv_moe_plan": (_i, [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _i64, _vp, _i64, _i, _i, _vp]),

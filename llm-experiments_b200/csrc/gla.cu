@@ -145,6 +145,13 @@ int launch_step(const b2kv_gla_args& a, int32_t* dev_status, void* stream) {
 
 using namespace b2kv;
 
+static bool takes_chunks(int path, int dtype, int max_n) { return path == 2 || (path == 0 && dtype == B2KV_DTYPE_BF16 && max_n > 16); }
+
+extern "C" size_t b2kv_gla_workspace_bytes(int H, int dim, int vdim, int n_segments, int max_n, int dtype, int path) {
+    if (H <= 0 || dim <= 0 || vdim <= 0 || n_segments <= 0 || max_n <= 0 || !takes_chunks(path, dtype, max_n)) return 0;
+    return gla_chunked_workspace(H, dim, vdim, n_segments, max_n, dtype);
+}
+
 extern "C" int b2kv_gla(const b2kv_gla_args* args, int32_t* dev_status, void* stream) {
     if (args == nullptr) return B2KV_ERR_BAD_ARG;
     const b2kv_gla_args& a = *args;
@@ -156,7 +163,7 @@ extern "C" int b2kv_gla(const b2kv_gla_args* args, int32_t* dev_status, void* st
     if (a.q_col < 0 || a.k_col < 0 || a.v_col < 0 || a.g_col < 0 || a.ld_y < a.q_col + keys || a.ld_y < a.k_col + keys ||
         a.ld_y < a.v_col + values || a.ld_y < a.g_col + values || a.ld_alpha < keys || a.ld_out < values)
         return B2KV_ERR_BAD_ARG;
-    if (a.path == 2 || (a.path == 0 && a.dtype == B2KV_DTYPE_BF16 && a.max_n > 16)) {
+    if (takes_chunks(a.path, a.dtype, a.max_n)) {
         const int rc = gla_chunked(a, dev_status, stream);
         if (rc != B2KV_ERR_UNSUPPORTED || a.path == 2) return rc;
     }

@@ -9,6 +9,7 @@ namespace b2kv {
 
 // Tensor-core kernel for segments of a prompt (bf16); B2KV_ERR_UNSUPPORTED when the shape is not one it takes.
 int gla_chunked(const b2kv_gla_args& a, int32_t* dev_status, void* stream);
+size_t gla_chunked_workspace(int H, int dim, int vdim, int n_segments, int max_n, int dtype);  // 0: no such form
 
 namespace gla {
 

@@ -374,7 +374,8 @@ int linear_rows_tc(const b2kv_linear_args& a, int32_t* dev_status, void* stream)
     if (tune_get("matmul_splits") > 0) {
         while (p.splits * 2 <= std::min(std::min(tune_get("matmul_splits"), 8), n_k)) p.splits *= 2;
     } else {
-        while (p.splits < 8 && tiles * p.splits * 2 <= 148 && n_k / (p.splits * 2) >= 2) p.splits *= 2;
+        // (clusters of eight find few places: they pay only where there are few of them)
+        while (p.splits < 8 && tiles * p.splits * 2 <= (p.splits == 4 ? 64 : 148) && n_k / (p.splits * 2) >= 2) p.splits *= 2;
     }
     while ((1 << p.split_shift) < p.splits) ++p.split_shift;
     const int recv_bytes = p.splits > 1 ? p.Bn * kFeat * 4 : 0;

@@ -45,11 +45,16 @@ def gated_linear_attention(ctx: GPUContext, y: GPUBuffer2D, cols: Tuple[int, int
         raise ValueError("the state does not have this layer's sizes")
     if alpha.buffer.dtype != torch.float32 or out.buffer.dtype != y.buffer.dtype or norm.buffer.dtype != torch.float32:
         raise ValueError("gated_linear_attention: alpha and norm are float32, out has the type of y")
+    dt = dtype_code(y.buffer.dtype)
+    nbytes = _native.lib.b2kv_gla_workspace_bytes(shape.heads, shape.dim, shape.vdim, segments.count, segments.max_n, dt, path)
+    if nbytes and (ctx.recurrent_workspace is None or ctx.recurrent_workspace.numel() < nbytes):
+        ctx.recurrent_workspace = torch.empty(nbytes, dtype=torch.uint8, device=ctx.device)
     a = _native.GlaArgs(
         y=y.buffer.data_ptr(), alpha=alpha.buffer.data_ptr(), norm=norm.buffer.data_ptr(), state=state.data_ptr(), out=out.buffer.data_ptr(),
-        segments=None if segments.table is None else segments.table.data_ptr(), row_pos=pos.data_ptr(), ld_y=y.buffer.stride(0),
+        segments=None if segments.table is None else segments.table.data_ptr(), row_pos=pos.data_ptr(),
+        workspace=ctx.recurrent_workspace.data_ptr() if nbytes else None, workspace_bytes=nbytes, ld_y=y.buffer.stride(0),
         ld_alpha=alpha.buffer.stride(0), ld_out=out.buffer.stride(0), q_col=cols[0], k_col=cols[1], v_col=cols[2], g_col=cols[3],
         H=shape.heads, dim=shape.dim, vdim=shape.vdim, n_segments=segments.count, max_n=segments.max_n, rows=y.shape[0],
-        n_slots=state.shape[0], dtype=dtype_code(y.buffer.dtype), path=path, q_scale=shape.dim ** -0.5, eps=eps)
+        n_slots=state.shape[0], dtype=dt, path=path, q_scale=shape.dim ** -0.5, eps=eps)
     stream = batch_op_begin(ctx)
     _native.check(_native.lib.b2kv_gla(ctypes.byref(a), dev_status_ptr(ctx), stream))

@@ -116,6 +116,7 @@ class GPUContext:
     dev_status: Optional[torch.Tensor] = None  # int32[1], written by kernels that detect a bad index
     perf_monitor: Optional[PerfMonitor] = None  # filled by batches opened with enable_profiling
     prefill_workspace: Optional[torch.Tensor] = None  # scratch of flash_attention for fp32 prompts, grown on demand
+    recurrent_workspace: Optional[torch.Tensor] = None  # scratch of recurrent layers over prompt portions, grown on demand
 
 
 @dataclass
