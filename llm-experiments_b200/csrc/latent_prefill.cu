@@ -20,7 +20,10 @@
 //     through.  K(j + 1) and V(j + 1) are then on their way while K(j) and V(j) are in use.
 //
 // Grouped heads (no rotated part) read the caches in place: key row t of a segment is a cache row, head h takes the columns of
-// key / value head h / (H / G).  A distance bias, slope_h * (query position - key position), is taken off the scores in fp32.
+// key / value head h / (H / G).  A distance bias, slope_h * (query position - key position), is taken off the scores in fp32
+// without work per score: the part that depends on the key's place in its tile, 0 ... 127, is one more k-step of the score product
+// (key rows hold their place, query rows slope / scale in three bf16 pieces, so the products are exact), the rest is a
+// constant of the row and the tile.
 //
 // TMEM columns: S_A 0-127, S_B 128-255, O_A 256-383, O_B 384-511.  Every wait is bounded.
 #include <math.h>
@@ -57,13 +60,14 @@ struct Params {
 };
 
 // kNope chunks per key, with kRot one more for the rotated part; kV chunks per value.
-template <int kNope, bool kRot, int kV>
+template <int kNope, bool kRot, int kV, bool kBias>
 struct Storage {
     static constexpr int kK = kNope + (kRot ? 1 : 0);
     static constexpr bool kSharedRing = kK == 3 && kV == 2;
     static constexpr int kChunks = kSharedRing ? 8 : 2 * (kK + kV);
     alignas(1024) uint8_t q[2][kK][kChunkBytes];
     alignas(1024) uint8_t kv[kChunks][kChunkBytes];
+    uint8_t ext[kBias ? kChunkBytes : 16];  // the bias's k-step: elements 0-15 of the key rows, 16-31 of the query rows
     alignas(8) uint64_t q_full;
     uint64_t k_full[2], k_empty[2], v_full[2], v_empty[2];
     uint64_t s_full[2], p_ready[2], o_done[2];
@@ -87,7 +91,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
                       const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
                       const __grid_constant__ CUtensorMap tm_v, const Params p) {
     extern __shared__ uint8_t smem_raw[];
-    using Smem = Storage<kNope, kRot, kV>;
+    using Smem = Storage<kNope, kRot, kV, kBias>;
     constexpr int kK = Smem::kK;
     Smem& sm = *reinterpret_cast<Smem*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -137,6 +141,21 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
     if (warp == 9) {
         tmem_alloc(&sm.tmem_base, kTmemCols);
         tmem_relinquish();
+    }
+    if (kBias && threadIdx.x < kBlockN) {
+        const float whole = p.slopes[h] * 1.4426950408889634f / p.prescale;  // slope / scale
+        const float hi = __bfloat162float(__float2bfloat16_rn(whole));
+        const float mid = __bfloat162float(__float2bfloat16_rn(whole - hi));
+        const float place = static_cast<float>(threadIdx.x);
+        uint4 piece[4] = {};
+        piece[0].x = pack_bf16(place, place);
+        piece[0].y = pack_bf16(place, 0.f);
+        piece[2].x = pack_bf16(hi, mid);
+        piece[2].y = pack_bf16(whole - hi - mid, 0.f);
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+            *reinterpret_cast<uint4*>(sm.ext + threadIdx.x * 128 + ((c ^ (threadIdx.x & 7)) << 4)) = piece[c];
+        fence_proxy_async_smem();
     }
     tc_fence_before();
     __syncthreads();
@@ -188,6 +207,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
             const uint64_t dq0 = smem_desc(smem_u32(sm.q[0][0]), 16, 1024), dq1 = smem_desc(smem_u32(sm.q[1][0]), 16, 1024);
             const uint64_t dk = smem_desc(smem_u32(sm.kv[0]), 16, 1024);
             const uint64_t dv = smem_desc(smem_u32(sm.kv[0]), kChunkBytes, 1024);
+            const uint64_t d_ext = smem_desc(smem_u32(sm.ext), 16, 1024);
             constexpr uint32_t kChunk16 = kChunkBytes >> 4;
             auto issue_qk = [&](int x, int j) {
                 const uint64_t a = x ? dq1 : dq0;
@@ -202,6 +222,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
                                kRot && c == kNope ? b_last + static_cast<uint64_t>(2 * kk) : b + static_cast<uint64_t>(c * kChunk16 + 2 * kk),
                                idesc_qk, (c | kk) ? 1u : 0u);
                 }
+                if (kBias) mma_ss(s_tmem, d_ext + static_cast<uint64_t>(2), d_ext, idesc_qk, 1u);
                 mma_commit(&sm.s_full[x]);
             };
             auto issue_pv = [&](int x, int j, bool first) {
@@ -281,21 +302,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
             const int hi = own + row - key0;
             const int lo = p.window > 0 ? hi - p.window + 1 : -1;
             const float2 c2 = make_float2(c, c);
-            if (kBias) {
-                // element e is hi - e tokens behind the query; four pairs of biases go along, eight elements at a step
-                float2 b[4];
-#pragma unroll
-                for (int a = 0; a < 4; ++a) b[a] = make_float2(slope * static_cast<float>(2 * a - hi), slope * static_cast<float>(2 * a + 1 - hi));
-                const float2 step = make_float2(8.f * slope, 8.f * slope);
-#pragma unroll
-                for (int e = 0; e < 128; e += 2) {
-                    float2& be = b[(e >> 1) & 3];
-                    const float2 z = __ffma2_rn(make_float2(__uint_as_float(r[e]), __uint_as_float(r[e + 1])), c2, be);
-                    be = __fadd2_rn(be, step);
-                    r[e] = __float_as_uint(z.x);
-                    r[e + 1] = __float_as_uint(z.y);
-                }
-            }
+            const float shift = kBias ? -slope * static_cast<float>(hi) : 0.f;  // what the row and the tile take off
             if (key0 + kBlockN - 1 > own || (p.window > 0 && own + kTileM - 1 - p.window + 1 > key0)) {
 #pragma unroll
                 for (int e = 0; e < 128; ++e)
@@ -308,7 +315,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
             for (int e = 8; e < 128; ++e) mxs[e & 7] = fmaxf(mxs[e & 7], __uint_as_float(r[e]));
             const float mx = fmaxf(fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3])),
                                    fmaxf(fmaxf(mxs[4], mxs[5]), fmaxf(mxs[6], mxs[7])));
-            m_run = fmaxf(m_run, kBias ? mx : mx * c);
+            m_run = fmaxf(m_run, kBias ? fmaf(mx, c, shift) : mx * c);
             float factor = 1.f;
             bool need = false;
             if (i == 0) {
@@ -318,7 +325,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
                 m_used = m_run;
                 need = true;
             }
-            const float neg_m = -m_used;
+            const float neg_m = shift - m_used;
             __syncwarp();  // the tensor-memory instructions below need the whole warp together
             float sums[8];
 #pragma unroll
@@ -330,7 +337,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
 #pragma unroll
                 for (int e = 0; e < 16; ++e) {
                     const float2 s2 = make_float2(__uint_as_float(r[cc * 32 + 2 * e]), __uint_as_float(r[cc * 32 + 2 * e + 1]));
-                    const float2 z = kBias ? __fadd2_rn(s2, neg_m2) : __ffma2_rn(s2, c2, neg_m2);
+                    const float2 z = __ffma2_rn(s2, c2, neg_m2);
                     const float p0 = ex2(z.x), p1 = ex2(z.y);
                     sums[(2 * e) & 7] += p0;
                     sums[(2 * e + 1) & 7] += p1;
@@ -416,7 +423,7 @@ static bool make_map(CUtensorMap* map, const void* base, int width, int heads, i
 
 template <int kNope, bool kRot, int kV, bool kBias>
 static int launch(const CUtensorMap (&m)[5], const Params& p, long long ctas, void* stream) {
-    constexpr size_t smem = sizeof(Storage<kNope, kRot, kV>) + 1024;
+    constexpr size_t smem = sizeof(Storage<kNope, kRot, kV, kBias>) + 1024;
     static_assert(smem <= 227 * 1024, "the tiles must fit one SM's shared memory");
     auto kernel = latent_prefill_kernel<kNope, kRot, kV, kBias>;
     static bool configured[64] = {false};
