@@ -1368,6 +1368,7 @@ def run_bamasun(h: Harness, w):
     and values attended, the states read and written) or whole prompts (prompt tokens/s, tensor roofline), and every kernel of
     the design timed alone on the model's own buffers."""
     torch, gpu, ctx = h.torch, h.gpu, h.ctx
+    from llm_experiments_b200 import _native as gpu_native
     from llm_experiments_b200 import bamasun, gqa, latent, recurrent
     from llm_experiments_b200.projection import SEG_DECAY, SEG_F32, SEG_RELU2, SEG_SOFTCAP, SEG_STORE, OutputSegment, linear
     from llm_experiments_b200.serving import RowSegments
@@ -1450,7 +1451,9 @@ def run_bamasun(h: Harness, w):
         nbytes = n_att * kv_bytes + n_gla * rows * state_bytes + 2 * (params + width * V)
     else:
         flops = 2.0 * rows * params + n_att * 2.0 * pairs * (a.dim + a.vdim) + n_gla * 4.0 * rows * g.heads * g.dim * g.vdim + 2.0 * B * width * V
-    launches = 9 * n_att + 8 * n_gla + 5 if decode else 8 * (n_att + n_gla) + 3
+    scratch = lambda n: gpu_native.lib.b2kv_gla_workspace_bytes(g.heads, g.dim, g.vdim, B, n, gpu_native.DTYPE_BF16, 2)  # noqa: E731
+    slices = 0 if decode else -(-(w["N"] // 16) * scratch(16) // scratch(w["N"]))  # of the chunked recurrence, two launches each
+    launches = 9 * n_att + 8 * n_gla + 5 if decode else 8 * n_att + (7 + 2 * slices) * n_gla + 3
     return run.record(measured, launches, clocks, nbytes, flops)
 
 

@@ -33,7 +33,7 @@ struct Piece<4> {
 };
 
 template <typename T, int kVec>
-__global__ void __launch_bounds__(kThreads) gla_step_kernel(const b2kv_gla_args a, int cx_count, int32_t* dev_status) {
+__global__ void __launch_bounds__(kThreads, 3) gla_step_kernel(const b2kv_gla_args a, int cx_count, int32_t* dev_status) {
     extern __shared__ float sm[];
     __shared__ float red[kThreads / 32];
     grid_launch_dependents();
