@@ -92,7 +92,7 @@ def state_close(state, want, rtol=1e-4):
 
 
 CASES = [(STEP, F32, 3, 5, 7), (STEP, BF, 2, 9, 33), (STEP, F32, 2, 48, 300), (STEP, BF, 4, 128, 256),
-         (CHUNK, BF, 4, 48, 32), (CHUNK, BF, 1, 8, 8), (CHUNK, BF, 3, 24, 72), (CHUNK, BF, 2, 64, 160), (CHUNK, BF, 2, 128, 256),
+         (CHUNK, BF, 5, 40, 24), (CHUNK, BF, 1, 8, 8), (CHUNK, BF, 3, 24, 72), (CHUNK, BF, 2, 64, 160), (CHUNK, BF, 2, 128, 256),
          (CHUNK, BF, 2, 104, 104), (CHUNK, BF, 3, 128, 64)]
 
 
@@ -109,7 +109,7 @@ def test_whole_sequences(pkg, path, dtype, heads, dim, vdim, n):
     assert torch.isnan(state[0]).all()
 
 
-@pytest.mark.parametrize("path,dtype,heads,dim,vdim", [(STEP, F32, 3, 5, 7), (CHUNK, BF, 4, 48, 40), (0, BF, 2, 128, 128), (0, BF, 2, 64, 64)])
+@pytest.mark.parametrize("path,dtype,heads,dim,vdim", [(STEP, F32, 3, 5, 7), (CHUNK, BF, 5, 56, 40), (0, BF, 2, 128, 128), (0, BF, 2, 64, 64)])
 def test_portions_carry_the_state(pkg, path, dtype, heads, dim, vdim):
     """Any cut gives the outputs of the whole, with two sequences in unequal portions per call and the rows of a call in any
     order; both kernels take turns when the choice is left open."""

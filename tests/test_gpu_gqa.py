@@ -119,7 +119,7 @@ def test_append_refuses_positions_outside_the_cache(pkg):
 
 
 SHAPES = [(SIMT, F32, 3, 1, 5, 7), (SIMT, BF, 4, 4, 9, 6), (SIMT, F32, 6, 2, 72, 130), (SIMT, F32, 2, 1, 300, 20),
-          (TC, BF, 8, 1, 48, 48), (TC, BF, 4, 4, 8, 128), (TC, BF, 10, 2, 128, 128), (TC, BF, 6, 1, 72, 40), (TC, BF, 40, 2, 64, 72),
+          (TC, BF, 7, 1, 56, 40), (TC, BF, 4, 4, 8, 128), (TC, BF, 10, 2, 128, 128), (TC, BF, 6, 1, 72, 40), (TC, BF, 40, 2, 64, 72),
           (TC, BF, 17, 1, 128, 64), (TC, BF, 70, 2, 24, 24)]
 
 
@@ -200,7 +200,7 @@ def test_a_single_key_among_hundreds_is_found(pkg, path, dtype):
         torch.testing.assert_close(out[r].double(), want, rtol=1e-2, atol=1e-2)
 
 
-@pytest.mark.parametrize("heads,kv,dim,vdim", [(8, 1, 48, 48), (6, 3, 128, 128), (4, 4, 72, 40), (5, 1, 64, 104), (2, 2, 8, 8)])
+@pytest.mark.parametrize("heads,kv,dim,vdim", [(7, 1, 56, 40), (6, 3, 128, 128), (4, 4, 72, 40), (5, 1, 64, 104), (2, 2, 8, 8)])
 @pytest.mark.parametrize("bias", [False, True])
 def test_prompt_portions(pkg, heads, kv, dim, vdim, bias):
     """Several sequences' portions in one launch: from the start, behind a cached part, across tile borders, of two rows."""
